@@ -324,20 +324,75 @@ def scaled_add_rmsnorm(x, y1, s1, y2, s2, weight, eps, out_dtype, rows=None, cop
     return res.to(out_dtype)
 
 
-def _rotate_half(v, cos_t, sin_t, rot):
+def _rotate(v, cos_t, sin_t, rot, interleaved=False):
     half = rot // 2
     r = v.clone()
     for i in range(half):
-        r[..., i] = v[..., i] * cos_t[i] - v[..., i + half] * sin_t[i]
-        r[..., i + half] = v[..., i + half] * cos_t[i] + v[..., i] * sin_t[i]
+        a, b = (2 * i, 2 * i + 1) if interleaved else (i, i + half)
+        r[..., a] = v[..., a] * cos_t[i] - v[..., b] * sin_t[i]
+        r[..., b] = v[..., b] * cos_t[i] + v[..., a] * sin_t[i]
     return r
 
 
+def embed_bigram(table, bigram, tokens, positions, tok_seq, cu_q, state, state_slots, mul_prev, mul_cur, scale=1.0, status=None):
+    """table[token] * scale + bigram[(previous * mul_prev + token * mul_cur) mod buckets], the last row at position 0."""
+    buckets = bigram.shape[0] - 1
+    out = embed(table, tokens, scale=scale)
+    for s in range(cu_q.numel() - 1):
+        r0, r1 = int(cu_q[s]), int(cu_q[s + 1])
+        if r1 == r0:
+            continue
+        slot = int(state_slots[s])
+        prev = int(state[slot, 0]) if int(positions[r0]) > 0 else None
+        for r in range(r0, r1):
+            cur = int(tokens[r])
+            out[r] += _f(bigram[buckets if prev is None else (prev * mul_prev + cur * mul_cur) % buckets])
+            prev = cur
+        state[slot, 0] = prev
+    return out
+
+
+def shift_add_rmsnorm(x, y1, s1, y2, s2, weight, eps, shift, state, state_slots, tok_seq, cu_q, positions, out_dtype, plain=True,
+                      status=None):
+    """v = x + s1 * y1 + s2 * y2;  h = rms(v) * weight;  shifted_t = h_t + (h_{t-1} - h_t) * shift.  Returns (v, h, shifted)."""
+    v = x
+    for y, sc in ((y1, s1), (y2, s2)):
+        if y is not None:
+            v = v + _f(y) * (sc if sc is not None else 1.0)
+    h = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * weight
+    shifted = torch.zeros_like(h)
+    W = h.shape[1]
+    for s in range(cu_q.numel() - 1):
+        r0, r1 = int(cu_q[s]), int(cu_q[s + 1])
+        if r1 == r0:
+            continue
+        slot = int(state_slots[s])
+        prev = state[slot, :W].clone() if int(positions[r0]) > 0 else torch.zeros(W)
+        for r in range(r0, r1):
+            shifted[r] = h[r] + (prev - h[r]) * shift
+            prev = h[r]
+        state[slot, :W] = prev
+    return v, h.to(out_dtype) if plain else None, shifted.to(out_dtype)
+
+
+def xielu(z, consts):
+    """up z^2 + z/2 above zero, down (exp(z) - 1 - z) + z/2 below; consts = [up, down]."""
+    v = _f(z)
+    low = torch.clamp(v, max=0.0)
+    return torch.where(v > 0, consts[0] * v * v + 0.5 * v, consts[1] * (torch.expm1(low) - low) + 0.5 * v).to(z.dtype)
+
+
+def linear_xielu(x, weight, consts):
+    return xielu(linear(x, weight, None, torch.float32), consts).to(x.dtype)
+
+
 def latent_prepare(down, q_rank, kv_rank, rot_dim, q_weight, kv_weight, eps, cos, sin, rot, cache_layer, page_size,
-                   slot_mapping, out_dtype, status=None):
+                   slot_mapping, out_dtype, status=None, interleaved=False, q=None, qfull=None, heads=0, dim=0):
     """down [n, q_rank | kv_rank | rot_dim] float32: the query latent normed; latent normed | key part rotated, into the page."""
     n = down.shape[0]
     cq = None
+    if q is not None:
+        latent_rotate_q(q, qfull, heads, dim, rot_dim, kv_rank, cos, sin, rot, interleaved)
     if q_rank > 0:
         a = down[:, :q_rank]
         cq = (a * torch.rsqrt(a.pow(2).mean(-1, keepdim=True) + eps) * q_weight).to(out_dtype)
@@ -348,20 +403,20 @@ def latent_prepare(down, q_rank, kv_rank, rot_dim, q_weight, kv_weight, eps, cos
             c = c * torch.rsqrt(c.pow(2).mean() + eps) * kv_weight
             kr = down[t, q_rank + kv_rank:q_rank + width]
             if rot > 0:
-                kr = _rotate_half(kr, cos[t], sin[t], rot)
+                kr = _rotate(kr, cos[t], sin[t], rot, interleaved)
             slot = int(slot_mapping[t])
             pg, off = slot // page_size, slot % page_size
             cache_layer[pg, off * width:(off + 1) * width] = torch.cat([c, kr]).to(cache_layer.dtype)
     return cq
 
 
-def latent_rotate_q(q, qfull, heads, dim, rot_dim, kv_rank, cos, sin, rot):
+def latent_rotate_q(q, qfull, heads, dim, rot_dim, kv_rank, cos, sin, rot, interleaved=False):
     n = q.shape[0]
     q3 = _f(q).view(n, heads, dim + rot_dim)
     for t in range(n):
         part = q3[t, :, dim:]
         if rot > 0:
-            part = _rotate_half(part, cos[t], sin[t], rot)
+            part = _rotate(part, cos[t], sin[t], rot, interleaved)
         qfull[t, :, kv_rank:] = part.to(qfull.dtype)
 
 
@@ -375,13 +430,13 @@ def head_products(x, w, out=None):
 
 
 def latent_attention(q, cache_layer, page_size, block_table, cu_q, seqlens_k, n, num_seqs, max_q, max_k, heads, kv_rank, rot_dim,
-                     scale, *, splits=None, status=None):
+                     scale, *, splits=None, status=None, sinks=None):
     width = kv_rank + rot_dim
     return masked_attention(q, heads * width, cache_layer, page_size, block_table, cu_q, seqlens_k, n, num_seqs, max_q, max_k,
-                            heads, 1, width, kv_rank, scale, shared_kv=True)
+                            heads, 1, width, kv_rank, scale, shared_kv=True, sinks=sinks)
 
 
-def gated_group_rmsnorm(y, z, weight, eps, group, gate_first, out_dtype, gate="silu"):
+def gated_group_rmsnorm(y, z, weight, eps, group, gate_first, out_dtype, gate="silu", out=None):
     n, width = y.shape
     zf = _f(z)
     gate = torch.sigmoid(zf) if gate == "sigmoid" else zf / (1.0 + torch.exp(-zf))
@@ -389,7 +444,11 @@ def gated_group_rmsnorm(y, z, weight, eps, group, gate_first, out_dtype, gate="s
     v = y * gate if gate_first else y
     v = v.view(n, width // group, group)
     v = (v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)).view(n, width) * w
-    return (v if gate_first else v * gate).to(out_dtype)
+    res = (v if gate_first else v * gate).to(out_dtype)
+    if out is None:
+        return res
+    out.copy_(res)
+    return out
 
 
 def scale_rows(x, factor):
@@ -450,9 +509,11 @@ def masked_attention_splits(num_seqs, max_q, max_k, nh, nkv):
 
 def masked_attention(q, q_row_stride, cache_layer, page_size, block_table, cu_q, seqlens_k, n, num_seqs, max_q, max_k,
                      nh, nkv, dk, dv, scale, *, window=0, chunk=0, sinks=None, gate=None, splits=None, status=None, keep=0,
-                     shared_kv=False):
-    """shared_kv: a page holds key rows alone and a key's value is the first dv elements of its row."""
+                     shared_kv=False, weights="softmax", softcap=0.0, score_bias=None, out_scale=1.0, out=None):
+    """shared_kv: a page holds key rows alone and a key's value is the first dv elements of its row.  softcap, then a bias
+    per head; weights "sigmoid": nothing is normalised over the keys."""
     rep = nh // nkv
+    given = out
     out = torch.zeros((n, nh * dv), dtype=torch.float32)
     kpart = nkv * page_size * dk
     for s in range(num_seqs):
@@ -474,6 +535,15 @@ def masked_attention(q, q_row_stride, cache_layer, page_size, block_table, cu_q,
                     else:
                         vs.append(_f(cache_layer[pg, kpart + (g * page_size + off) * dv:kpart + (g * page_size + off + 1) * dv]))
                 sc = torch.stack(ks) @ qv * scale
+                if softcap > 0:
+                    sc = softcap * torch.tanh(sc / softcap)
+                if score_bias is not None:
+                    sc = sc + score_bias[h]
+                if weights == "sigmoid":
+                    out[q0 + j, h * dv:(h + 1) * dv] = torch.sigmoid(sc) @ torch.stack(vs) * out_scale
+                    if gate is not None:
+                        out[q0 + j, h * dv:(h + 1) * dv] *= torch.sigmoid(_f(gate[q0 + j, h]))
+                    continue
                 mx = sc.max()
                 if sinks is not None:
                     mx = torch.maximum(mx, sinks[h])
@@ -482,7 +552,10 @@ def masked_attention(q, q_row_stride, cache_layer, page_size, block_table, cu_q,
                 o = (e / den) @ torch.stack(vs)
                 if gate is not None:
                     o = o * torch.sigmoid(_f(gate[q0 + j, h]))
-                out[q0 + j, h * dv:(h + 1) * dv] = o
+                out[q0 + j, h * dv:(h + 1) * dv] = o * out_scale
+    if given is not None:
+        given.copy_(out.to(q.dtype))
+        return given
     return out.to(q.dtype)
 
 
@@ -796,4 +869,4 @@ ALL = ["matrix_memory", "gated_linear_attention", "embed", "resolve_tokens", "sa
        "qk_norm_rope_write_split", "masked_attention_splits", "masked_attention", "causal_conv_silu", "gated_delta",
        "state_space", "causal_conv", "embed_sinusoid", "hyper_read_norm", "branch_rmsnorm_mean", "sigmoid_gate", "softcap",
        "rglru", "relu_squared", "moe_route", "moe_experts", "moe_table_route", "scaled_add_rmsnorm", "latent_prepare",
-       "latent_rotate_q", "head_products", "latent_attention"]
+       "latent_rotate_q", "head_products", "latent_attention", "embed_bigram", "shift_add_rmsnorm", "xielu", "linear_xielu"]

@@ -9,7 +9,8 @@
 // pairs (one kv head: all heads of a token share the keys), cut into tiles of 64; a block of four warps takes one tile,
 // a warp 16 rows of it; keys are walked in tiles of 64 through two shared-memory stages of 16-byte cp.async copies (rows
 // padded by 16 bytes, which makes ldmatrix conflict-free when dk is a multiple of 16); keys no row can see are stored as
-// zeros, so uninitialised cache memory never reaches the arithmetic.  mma.sync m16n8k16, float accumulators; scores,
+// zeros, so uninitialised cache memory never reaches the arithmetic.  A learned sink per head may join the softmax's
+// denominator (counted by the first split).  mma.sync m16n8k16, float accumulators; scores,
 // mask, running maximum and sum in float registers; P is rounded to bfloat16 only as the operand of P.V.  With splits >
 // 1 the key tiles are divided among blocks that leave partial results for the fixed-order combine of
 // attention_masked.cu.
@@ -41,7 +42,7 @@ latent_flash_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
                     const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_q,
                     const int* __restrict__ seqlens_k, __nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
                     float* __restrict__ part_ml, int nh, int dk, int dv, int page_size, int num_pages, float scale,
-                    int splits, int* __restrict__ status) {
+                    int splits, int* __restrict__ status, const float* __restrict__ sinks) {
     extern __shared__ __align__(128) unsigned char lf_smem[];
     const int ldk = dk + 8;                                            // elements; rows stay 16-byte aligned
     __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(lf_smem);     // [LF_ROWS][ldk]
@@ -241,6 +242,16 @@ latent_flash_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
         const int rr = tile_start + warp * 16 + gq + 8 * h2;
         const int tok = rr / nh, h = rr - tok * nh;
         const size_t grow = (size_t)(q0 + tok) * nh + h;
+        if (sinks && sp == 0) {
+            // the sink joins as one more term of the denominator, with no value (the running maximum is in base 2)
+            const float sk = sinks[h] * 1.4426950408889634f;
+            const float m_new = fmaxf(m[h2], sk);
+            const float alpha2 = m[h2] == -INFINITY ? 0.f : exp2f(m[h2] - m_new);
+            l[h2] = l[h2] * alpha2 + exp2f(sk - m_new);
+            m[h2] = m_new;
+#pragma unroll
+            for (int i = 0; i < NTV; ++i) { o[i][2 * h2] *= alpha2; o[i][2 * h2 + 1] *= alpha2; }
+        }
         if (splits == 1) {
             const float inv = l[h2] > 0.f ? 1.f / l[h2] : 0.f;
 #pragma unroll
@@ -273,7 +284,7 @@ inline bool latent_flash_applies(int dk, int dv, long long q_row_stride, const v
 static int launch_latent_flash(const void* q, long long q_row_stride, const void* cache, const int* block_table, int table_stride,
                                const int* cu_q, const int* seqlens_k, void* out, float* part_o, float* part_ml, int num_seqs,
                                int max_q, int nh, int dk, int dv, int page_size, int num_pages, float scale, int splits,
-                               int* status, cudaStream_t stream) {
+                               int* status, cudaStream_t stream, const float* sinks = nullptr) {
     const size_t smem = (size_t)(LF_ROWS + 2 * LF_BK) * (dk + 8) * sizeof(__nv_bfloat16);
     const int tiles = (int)(((long long)max_q * nh + LF_ROWS - 1) / LF_ROWS);
     if ((long long)num_seqs * splits > 65535) return fail(-1, "latent attention: %d sequences in %d splits", num_seqs, splits);
@@ -290,7 +301,7 @@ static int launch_latent_flash(const void* q, long long q_row_stride, const void
         }                                                                                                                      \
         e = launch(kern, grid, LF_THREADS, smem, stream, (const __nv_bfloat16*)q, q_row_stride, (const __nv_bfloat16*)cache,   \
                    block_table, table_stride, cu_q, seqlens_k, (__nv_bfloat16*)out, part_o, part_ml, nh, dk, dv, page_size,    \
-                   num_pages, scale, splits, status);                                                                          \
+                   num_pages, scale, splits, status, sinks);                                                                          \
     } while (0)
     if (dv <= 64) LF_GO(8);
     else if (dv <= 128) LF_GO(16);

@@ -9,7 +9,10 @@
 // sequence that a window never leaves behind)  and  floor(i / chunk) = floor(p / chunk)
 // (chunk > 0; chunks are counted from position 0 of the sequence).  score = scale * q.k; the
 // softmax's denominator also holds exp(sink_h) when sinks are given (no key, no value, unscaled);
-// head h's output is multiplied by sigmoid(gate[token, h]) when a gate is given.
+// head h's output is multiplied by sigmoid(gate[token, h]) when a gate is given.  Other forms of the weights
+// (ScoreForm in attention_mma.cuh): scores may pass a soft cap, a number per head may be added to them, and a visible
+// key's weight may be the sigmoid of its score with nothing normalised over the keys; the output may be multiplied by
+// a number and may go into rows of a wider buffer.
 //
 // A cache page holds the keys [nkv, page_size, dk] and then the values [nkv, page_size, dv].  With `shared_kv` a
 // page holds the key rows alone and a key's value is the first dv elements of its own row (latent attention: the
@@ -64,7 +67,7 @@ masked_attention_kernel(const T* __restrict__ q, long long q_row_stride, const T
                         const T* __restrict__ gate, long long gate_stride, T* __restrict__ out,
                         float* __restrict__ part_o, float* __restrict__ part_ml, int nh, int nkv, int dk, int dv,
                         int page_size, int num_pages, float scale, int window, int chunk, int splits,
-                        int* __restrict__ status, int keep, int shared_kv) {
+                        int* __restrict__ status, int keep, int shared_kv, const ScoreForm form) {
     constexpr int DPL = DVMAX / 32;
     extern __shared__ __align__(16) float smem[];
     const int ldk = dk + 4, ldv = dv + 4;
@@ -118,12 +121,14 @@ masked_attention_kernel(const T* __restrict__ q, long long q_row_stride, const T
 
     int row_pos[MA_RPW];
     bool row_ok[MA_RPW];
+    float row_bias[MA_RPW];
     float m[MA_RPW], l[MA_RPW], acc[MA_RPW][DPL];
 #pragma unroll
     for (int a = 0; a < MA_RPW; ++a) {
         const int rr = tile_start + warp + MA_WARPS * a;
         row_ok[a] = rr < rows_total;
         row_pos[a] = base_pos + (row_ok[a] ? rr / n_rep : 0);
+        row_bias[a] = (form.bias && row_ok[a]) ? form.bias[g * n_rep + rr % n_rep] : 0.f;
         m[a] = -INFINITY;
         l[a] = 0.f;
 #pragma unroll
@@ -183,6 +188,12 @@ masked_attention_kernel(const T* __restrict__ q, long long q_row_stride, const T
         for (int a = 0; a < MA_RPW; ++a) {
             if (!row_ok[a]) continue;
             const bool vis = ma_visible(j, row_pos[a], klen, window, chunk, keep);
+            if (form.softcap > 0.f) sc[a] = form.softcap * tanhf(sc[a] / form.softcap);
+            if (form.bias) sc[a] += row_bias[a];
+            if (form.sigmoid) {
+                pw[a * MA_BK + lane] = vis ? 1.f / (1.f + expf(-sc[a])) : 0.f;
+                continue;
+            }
             const float sv = vis ? sc[a] : -INFINITY;
             const float m_new = fmaxf(m[a], warp_max(sv));
             float p = 0.f, alpha = 1.f;
@@ -221,7 +232,7 @@ masked_attention_kernel(const T* __restrict__ q, long long q_row_stride, const T
         const int rr = tile_start + warp + MA_WARPS * a;
         const int tok = rr / n_rep, h = g * n_rep + (rr - tok * n_rep);
         const size_t grow = (size_t)(q0 + tok) * nh + h;
-        if (sinks && sp == 0) {
+        if (sinks && sp == 0 && !form.sigmoid) {
             // the sink joins as one more term of the denominator, with no value
             const float sk = sinks[h];
             const float m_new = fmaxf(m[a], sk);
@@ -232,12 +243,14 @@ masked_attention_kernel(const T* __restrict__ q, long long q_row_stride, const T
             for (int c = 0; c < DPL; ++c) acc[a][c] *= alpha;
         }
         if (splits == 1) {
-            float inv = l[a] > 0.f ? 1.f / l[a] : 0.f;
+            float inv = form.sigmoid ? 1.f : (l[a] > 0.f ? 1.f / l[a] : 0.f);
             if (gate) inv *= 1.f / (1.f + expf(-to_f32(gate[(size_t)(q0 + tok) * gate_stride + h])));
+            inv *= form.out_scale;
+            T* orow = out + (size_t)(q0 + tok) * form.out_stride + (size_t)h * dv;
 #pragma unroll
             for (int c = 0; c < DPL; ++c) {
                 const int col = lane + 32 * c;
-                if (col < dv) out[grow * dv + col] = from_f32<T>(acc[a][c] * inv);
+                if (col < dv) orow[col] = from_f32<T>(acc[a][c] * inv);
             }
         } else {
             float* po = part_o + (grow * splits + sp) * (size_t)dv;
@@ -258,7 +271,7 @@ masked_attention_kernel(const T* __restrict__ q, long long q_row_stride, const T
 template <typename T>
 __global__ void masked_attention_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                 const T* __restrict__ gate, long long gate_stride, T* __restrict__ out,
-                                                long long rows, int nh, int dv, int splits) {
+                                                long long rows, int nh, int dv, int splits, const ScoreForm form) {
     const long long row = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     pdl_trigger();
@@ -270,13 +283,15 @@ __global__ void masked_attention_combine_kernel(const float* __restrict__ part_o
         ls = part_ml[(row * splits + lane) * 2 + 1];
     }
     const float mx = warp_max(ms);
-    const float w = ms == -INFINITY ? 0.f : expf(ms - mx);
+    // weights that are not normalised over the keys simply add up
+    const float w = form.sigmoid ? 1.f : (ms == -INFINITY ? 0.f : expf(ms - mx));
     float lsum = 0.f;
     for (int sp = 0; sp < splits; ++sp) lsum += __shfl_sync(0xffffffffu, ls * w, sp);
-    float inv = lsum > 0.f ? 1.f / lsum : 0.f;
+    float inv = form.sigmoid ? 1.f : (lsum > 0.f ? 1.f / lsum : 0.f);
+    const long long tok = row / nh;
+    const int h = (int)(row - tok * nh);
+    inv *= form.out_scale;
     if (gate) {
-        const long long tok = row / nh;
-        const int h = (int)(row - tok * nh);
         inv *= 1.f / (1.f + expf(-to_f32(gate[(size_t)tok * gate_stride + h])));
     }
     for (int c0 = 0; c0 < dv; c0 += 32) {
@@ -287,7 +302,7 @@ __global__ void masked_attention_combine_kernel(const float* __restrict__ part_o
             const float v = col < dv ? part_o[(row * splits + sp) * (size_t)dv + col] : 0.f;
             o += v * ws;
         }
-        if (col < dv) out[row * dv + col] = from_f32<T>(o * inv);
+        if (col < dv) out[(size_t)tok * form.out_stride + (size_t)h * dv + col] = from_f32<T>(o * inv);
     }
 }
 
@@ -297,7 +312,7 @@ static int launch_masked(const void* q, long long q_row_stride, const void* cach
                          const void* gate, long long gate_stride, void* out, float* part_o, float* part_ml, int n,
                          int num_seqs, int max_q, int nh, int nkv, int dk, int dv, int page_size, int num_pages,
                          float scale, int window, int chunk, int splits, int* status, cudaStream_t stream, int keep,
-                         int shared_kv) {
+                         int shared_kv, const ScoreForm& form) {
     const int n_rep = nh / nkv;
     const int tiles = (max_q * n_rep + MA_ROWS - 1) / MA_ROWS;
     const size_t smem = sizeof(float) * ((size_t)(MA_ROWS + MA_BK) * (dk + 4) + (size_t)MA_BK * (dv + 4) +
@@ -313,12 +328,12 @@ static int launch_masked(const void* q, long long q_row_stride, const void* cach
     dim3 grid(tiles, nkv, num_seqs * splits);
     cudaError_t e = launch(kern, grid, MA_WARPS * 32, smem, stream, (const T*)q, q_row_stride, (const T*)cache, block_table,
                            table_stride, cu_q, seqlens_k, sinks, (const T*)gate, gate_stride, (T*)out, part_o, part_ml, nh, nkv,
-                           dk, dv, page_size, num_pages, scale, window, chunk, splits, status, keep, shared_kv);
+                           dk, dv, page_size, num_pages, scale, window, chunk, splits, status, keep, shared_kv, form);
     int rc = check_launch("masked_attention", e);
     if (rc != 0 || splits == 1) return rc;
     const long long rows = (long long)n * nh;
     e = launch(masked_attention_combine_kernel<T>, (int)((rows + 3) / 4), 128, 0, stream, (const float*)part_o,
-               (const float*)part_ml, (const T*)gate, gate_stride, (T*)out, rows, nh, dv, splits);
+               (const float*)part_ml, (const T*)gate, gate_stride, (T*)out, rows, nh, dv, splits, form);
     return check_launch("masked_attention_combine", e);
 }
 
@@ -328,8 +343,17 @@ VAPI_EXPORT int vapi_masked_attention(const void* q, long long q_row_stride, con
                                       long long gate_stride, void* out, float* part_o, float* part_ml, int n,
                                       int num_seqs, int max_q, int nh, int nkv, int dk, int dv, int page_size,
                                       int num_pages, float scale, int window, int chunk, int splits, int* status,
-                                      cudaStream_t stream, int keep, int shared_kv) {
+                                      cudaStream_t stream, int keep, int shared_kv, float softcap, int sigmoid,
+                                      const float* score_bias, float out_scale, long long out_stride) {
     if (n <= 0 || num_seqs <= 0) return 0;
+    ScoreForm form;
+    form.sigmoid = sigmoid ? 1 : 0;
+    form.softcap = softcap > 0.f ? softcap : 0.f;
+    form.bias = score_bias;
+    form.out_scale = out_scale;
+    form.out_stride = out_stride;
+    if (out_stride < (long long)nh * dv) return fail(-1, "masked_attention: output rows of %lld elements for %d heads of %d", out_stride, nh, dv);
+    if (sigmoid && sinks) return fail(-1, "masked_attention: a sink belongs to a softmax");
     if (shared_kv && dv > dk) return fail(-1, "masked_attention: values of %d inside key rows of %d", dv, dk);
     if (keep < 0) return fail(-1, "masked_attention: %d kept first tokens", keep);
     if (window <= 0) keep = 0;
@@ -340,52 +364,61 @@ VAPI_EXPORT int vapi_masked_attention(const void* q, long long q_row_stride, con
     if (splits < 1 || splits > 32) return fail(-1, "masked_attention: %d splits", splits);
     if (splits > 1 && (!part_o || !part_ml)) return fail(-1, "masked_attention: splits need scratch buffers");
     if (page_size <= 0 || num_pages <= 0) return fail(-1, "masked_attention: no pages");
+    // (the tensor-core kernels know the plain softmax and the sigmoid form; a capped or biased softmax runs below)
     if (!shared_kv && dtype == VAPI_BF16 && dk == dv && (dk == 64 || dk == 128) && page_size % FA_BK == 0 && q_row_stride % 2 == 0 &&
-        nkv <= 65535 && (long long)num_seqs * splits <= 65535) {
+        (form.sigmoid || form.plain()) && out_stride % 2 == 0 && ((uintptr_t)out & 3) == 0 && nkv <= 65535 && (long long)num_seqs * splits <= 65535) {
         // the cache page is [2][nkv][page_size][d] when keys and values have one width: the layout of the fast kernels
         int rc;
         const bool tc_ok = dk == FT_HD && splits == 1 && q_row_stride % 8 == 0 && scale > 0.f && max_q >= FT_AUTO_MAX_Q &&
-                           ((uintptr_t)q & 15) == 0 && ((uintptr_t)out & 15) == 0;
+                           ((uintptr_t)q & 15) == 0 && ((uintptr_t)out & 15) == 0 && out_stride % 8 == 0;
         if (tc_ok) {
             const int min_q = num_seqs == 1 ? 1 : FT_MIN_Q;
-            rc = launch_flash_tc(q, q_row_stride, cache, block_table, table_stride, cu_q, seqlens_k, out, num_seqs, max_q, nh,
-                                 nkv, page_size, num_pages, scale, window, min_q, status, stream, chunk, sinks, gate, gate_stride, keep);
-            if (rc != 0 || min_q == 1) return rc;
-            return launch_flash<64, 4, 3>(q, q_row_stride, cache, block_table, table_stride, cu_q, seqlens_k, out, part_o, part_ml,
-                                          num_seqs, FT_MIN_Q - 1, nh, nkv, page_size, num_pages, scale, window, 1, status, stream,
-                                          FT_MIN_Q, 0, chunk, sinks, gate, gate_stride, keep);
+#define MA_TC(SIG)                                                                                                            \
+    rc = launch_flash_tc<SIG>(q, q_row_stride, cache, block_table, table_stride, cu_q, seqlens_k, out, num_seqs, max_q, nh, nkv, \
+                              page_size, num_pages, scale, window, min_q, status, stream, chunk, sinks, gate, gate_stride, keep, \
+                              form);                                                                                          \
+    if (rc != 0 || min_q == 1) return rc;                                                                                     \
+    return launch_flash<64, 4, 3, SIG>(q, q_row_stride, cache, block_table, table_stride, cu_q, seqlens_k, out, part_o, part_ml, \
+                                       num_seqs, FT_MIN_Q - 1, nh, nkv, page_size, num_pages, scale, window, 1, status, stream, \
+                                       FT_MIN_Q, 0, chunk, sinks, gate, gate_stride, keep, form)
+            if (form.sigmoid) { MA_TC(true); }
+            MA_TC(false);
+#undef MA_TC
         }
         const bool few_rows = (long long)max_q * (nh / nkv) <= 16;
-#define MA_FLASH(HD, NW)                                                                                                      \
-    rc = launch_flash<HD, NW, 3>(q, q_row_stride, cache, block_table, table_stride, cu_q, seqlens_k, out, part_o, part_ml,    \
-                                 num_seqs, max_q, nh, nkv, page_size, num_pages, scale, window, splits, status, stream, 0, 0, \
-                                 chunk, sinks, gate, gate_stride, keep)
-        if (dk == 64) { if (few_rows) MA_FLASH(64, 1); else MA_FLASH(64, 4); }
-        else          { if (few_rows) MA_FLASH(128, 1); else MA_FLASH(128, 4); }
+#define MA_FLASH(HD, NW, SIG)                                                                                                      \
+    rc = launch_flash<HD, NW, 3, SIG>(q, q_row_stride, cache, block_table, table_stride, cu_q, seqlens_k, out, part_o, part_ml,    \
+                                      num_seqs, max_q, nh, nkv, page_size, num_pages, scale, window, splits, status, stream, 0, 0, \
+                                      chunk, sinks, gate, gate_stride, keep, form)
+#define MA_WIDTHS(SIG)                                                                     \
+    if (dk == 64) { if (few_rows) MA_FLASH(64, 1, SIG); else MA_FLASH(64, 4, SIG); }       \
+    else          { if (few_rows) MA_FLASH(128, 1, SIG); else MA_FLASH(128, 4, SIG); }
+        if (form.sigmoid) { MA_WIDTHS(true) } else { MA_WIDTHS(false) }
+#undef MA_WIDTHS
 #undef MA_FLASH
         if (rc != 0 || splits == 1) return rc;
         const long long rows = (long long)n * nh;
         return check_launch("masked_attention_combine",
                             launch(masked_attention_combine_kernel<__nv_bfloat16>, (int)((rows + 3) / 4), 128, 0, stream,
                                    (const float*)part_o, (const float*)part_ml, (const __nv_bfloat16*)gate, gate_stride,
-                                   (__nv_bfloat16*)out, rows, nh, dv, splits));
+                                   (__nv_bfloat16*)out, rows, nh, dv, splits, form));
     }
-    if (shared_kv && dtype == VAPI_BF16 && !sinks && !gate && window <= 0 && chunk <= 0 &&
-        latent_flash_applies(dk, dv, q_row_stride, q, cache, out)) {
+    if (shared_kv && dtype == VAPI_BF16 && form.plain() && out_scale == 1.f && out_stride == (long long)nh * dv && !gate &&
+        window <= 0 && chunk <= 0 && nkv == 1 && latent_flash_applies(dk, dv, q_row_stride, q, cache, out)) {
         // one cached row per token that is key and value at once: the tensor-core kernel of attention_latent.cuh
         int rc = launch_latent_flash(q, q_row_stride, cache, block_table, table_stride, cu_q, seqlens_k, out, part_o, part_ml,
-                                     num_seqs, max_q, nh, dk, dv, page_size, num_pages, scale, splits, status, stream);
+                                     num_seqs, max_q, nh, dk, dv, page_size, num_pages, scale, splits, status, stream, sinks);
         if (rc != 0 || splits == 1) return rc;
         const long long rows = (long long)n * nh;
         return check_launch("masked_attention_combine",
                             launch(masked_attention_combine_kernel<__nv_bfloat16>, (int)((rows + 3) / 4), 128, 0, stream,
                                    (const float*)part_o, (const float*)part_ml, (const __nv_bfloat16*)nullptr, (long long)0,
-                                   (__nv_bfloat16*)out, rows, nh, dv, splits));
+                                   (__nv_bfloat16*)out, rows, nh, dv, splits, form));
     }
 #define MA_GO(T, DV) return launch_masked<T, DV>(q, q_row_stride, cache, block_table, table_stride, cu_q, seqlens_k, sinks, gate, \
                                                  gate_stride, out, part_o, part_ml, n, num_seqs, max_q, nh, nkv, dk, dv,         \
                                                  page_size, num_pages, scale, window, chunk, splits, status, stream, keep,  \
-                                                 shared_kv)
+                                                 shared_kv, form)
     if (dtype == VAPI_F32) {
         if (dv <= 64) MA_GO(float, 64);
         if (dv <= 128) MA_GO(float, 128);

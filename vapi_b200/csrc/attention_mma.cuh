@@ -49,7 +49,89 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 
 constexpr int FA_BK = 64;
 
-template <int HD, int NWARPS, int STAGES>
+// How a score becomes a weight, beyond the plain softmax, and where the result goes.
+//   softcap > 0:  score <- softcap * tanh(score / softcap);   bias: a number per head is added to the score then
+//   sigmoid:      a visible key's weight is sigmoid(score), and nothing is normalised over the keys
+//   out_scale:    the head's output is multiplied by it (before its one rounding)
+//   out_stride:   elements between two tokens' output rows (0: heads * value width, i.e. contiguous)
+struct ScoreForm {
+    int sigmoid = 0;
+    float softcap = 0.f;
+    const float* bias = nullptr;
+    float out_scale = 1.f;
+    long long out_stride = 0;
+    bool plain() const { return !sigmoid && softcap <= 0.f && !bias; }
+};
+
+// The sigmoid form with its constants worked out for base-2 exponentials: with a raw product s = q.k,
+//   capped:  weight = 1 / (1 + 2^(kc * tanh(k1 * s) + nb)),  k1 = scale / cap, kc = -cap * log2 e
+//   else     weight = 1 / (1 + 2^(k1 * s + nb)),             k1 = -scale * log2 e
+// and nb = -bias[head] * log2 e, a row's own number.
+struct SigmoidForm { float k1 = 0.f, kc = 0.f; int capped = 0; };
+
+inline SigmoidForm sigmoid_form(float scale, float softcap) {
+    SigmoidForm f;
+    const float log2e = 1.4426950408889634f;
+    f.capped = softcap > 0.f;
+    f.k1 = f.capped ? scale / softcap : -scale * log2e;
+    f.kc = f.capped ? -softcap * log2e : 0.f;
+    return f;
+}
+
+__device__ __forceinline__ float ex2_ftz(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp_ftz(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// N raw products of one row -> their weights, in place.  Every lane of the warp must take part.  The products of normed
+// queries and keys usually stay far below the cap, so tanh is its odd Taylor polynomial while no lane's |k1 s| reaches
+// 0.3 (error below 2e-8) and 1 - 2 / (1 + e^2u) otherwise; two weights share one reciprocal, 1/a = b / (ab) (exponents
+// are clamped at 62, where a weight is below 2^-61, so that the product stays finite).
+template <int N>
+__device__ __forceinline__ void sigmoid_weights(float (&s)[N], const SigmoidForm& f, float nb) {
+    static_assert(N % 2 == 0, "weights come in pairs");
+    if (f.capped) {
+        float um = 0.f;
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            s[i] *= f.k1;
+            um = fmaxf(um, fabsf(s[i]));
+        }
+        if (!__any_sync(0xffffffffu, um >= 0.3f)) {
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                const float u = s[i], z = u * u;
+                const float t = fmaf(z, fmaf(z, fmaf(z, fmaf(z, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
+                s[i] = fmaf(u * t, f.kc, nb);
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                const float e = ex2_ftz(fminf(s[i] * 2.8853900817779268f, 126.f));
+                s[i] = fmaf(fmaf(-2.f, rcp_ftz(1.f + e), 1.f), f.kc, nb);
+            }
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) s[i] = fmaf(s[i], f.k1, nb);
+    }
+#pragma unroll
+    for (int i = 0; i < N; i += 2) {
+        const float a = 1.f + ex2_ftz(fminf(s[i], 62.f)), b = 1.f + ex2_ftz(fminf(s[i + 1], 62.f));
+        const float r = rcp_ftz(a * b);
+        s[i] = r * b;
+        s[i + 1] = r * a;
+    }
+}
+
+// SIG: weights are sigmoids of the scores (SigmoidForm), not normalised over the keys
+template <int HD, int NWARPS, int STAGES, bool SIG = false>
 __global__ void __launch_bounds__(NWARPS * 32, (HD <= 64 && NWARPS == 4) ? 4 : 1)
 flash_paged_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
                    const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_table,
@@ -58,7 +140,9 @@ flash_paged_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
                    float* __restrict__ part_ml, int nh, int nkv, int page_size, int num_pages,
                    float scale_log2e, int window, int splits, int q_below, int rows_above,
                    int* __restrict__ status, int mask_chunk = 0, const float* __restrict__ sinks = nullptr,
-                   const __nv_bfloat16* __restrict__ gate = nullptr, long long gate_stride = 0, int keep = 0) {
+                   const __nv_bfloat16* __restrict__ gate = nullptr, long long gate_stride = 0, int keep = 0,
+                   SigmoidForm sig = SigmoidForm(), const float* __restrict__ score_bias = nullptr, float out_scale = 1.f,
+                   long long out_stride = 0) {
     // keep > 0 (with a window): the first `keep` tokens of a sequence stay visible behind the window
     // mask_chunk > 0: a query also sees only keys of its own block of mask_chunk positions (counted from
     // position 0); sinks: exp(sink[head]) joins the softmax's denominator (counted by the first split);
@@ -132,6 +216,12 @@ flash_paged_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
     float o_acc[HD / 8][4];
 #pragma unroll
     for (int i = 0; i < HD / 8; ++i) { o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f; }
+
+    float nb[2] = {0.f, 0.f};                            // a row's share of the exponent (SIG)
+    if (SIG && score_bias) {
+        nb[0] = -1.4426950408889634f * score_bias[row_head[0]];
+        nb[1] = -1.4426950408889634f * score_bias[row_head[1]];
+    }
 
     const int* bt = block_table + (size_t)s * table_stride;
     const int key_hi = min(klen - 1, p_max);
@@ -231,8 +321,27 @@ flash_paged_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
         const bool need_mask = (k0 + FA_BK - 1 > w_pos_min) || (k0 + FA_BK > klen) ||
                                (window > 0 && k0 <= w_pos_max - window) ||
                                (mask_chunk > 0 && k0 < (w_pos_max / mask_chunk) * mask_chunk);
+        if (SIG) {
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
+            for (int h = 0; h < 2; ++h) {
+                float w16[16];
+#pragma unroll
+                for (int i = 0; i < 16; ++i) w16[i] = sc[i >> 1][2 * h + (i & 1)];
+                sigmoid_weights(w16, sig, nb[h]);
+#pragma unroll
+                for (int i = 0; i < 16; ++i) {
+                    if (need_mask) {
+                        const int kj = k0 + (i >> 1) * 8 + 2 * tq + (i & 1);
+                        const bool vis = kj <= row_pos[h] && kj < klen && (window <= 0 || kj > row_pos[h] - window || kj < keep) &&
+                                         kj >= row_lo[h];
+                        w16[i] = vis ? w16[i] : 0.f;
+                    }
+                    sc[i >> 1][2 * h + (i & 1)] = w16[i];
+                }
+            }
+        }
+#pragma unroll
+        for (int h = 0; h < (SIG ? 0 : 2); ++h) {
             float mx = -INFINITY;
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
@@ -298,7 +407,7 @@ flash_paged_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
         l += __shfl_xor_sync(0xffffffffu, l, 2);
         if (!row_ok[h]) continue;
         const size_t grow = (size_t)(q0 + row_tok[h]) * nh + row_head[h];
-        if (sinks && sp == 0) {
+        if (!SIG && sinks && sp == 0) {
             const float sk = sinks[row_head[h]] * 1.4426950408889634f;       // the running maximum is in base 2
             const float m_new = fmaxf(m_run[h], sk);
             const float alpha = m_run[h] == -INFINITY ? 0.f : exp2f(m_run[h] - m_new);
@@ -308,9 +417,10 @@ flash_paged_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
             for (int i = 0; i < HD / 8; ++i) { o_acc[i][2 * h] *= alpha; o_acc[i][2 * h + 1] *= alpha; }
         }
         if (splits == 1) {
-            float inv = l > 0.f ? 1.f / l : 0.f;
+            float inv = SIG ? 1.f : (l > 0.f ? 1.f / l : 0.f);
             if (gate) inv *= 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)(q0 + row_tok[h]) * gate_stride + row_head[h]])));
-            __nv_bfloat16* o = out + grow * HD;
+            inv *= out_scale;
+            __nv_bfloat16* o = out_stride > 0 ? out + (size_t)(q0 + row_tok[h]) * out_stride + (size_t)row_head[h] * HD : out + grow * HD;
 #pragma unroll
             for (int i = 0; i < HD / 8; ++i) {
                 __nv_bfloat162 v = __floats2bfloat162_rn(o_acc[i][2 * h] * inv, o_acc[i][2 * h + 1] * inv);
@@ -331,14 +441,14 @@ flash_paged_kernel(const __nv_bfloat16* __restrict__ q, long long q_row_stride,
     }
 }
 
-template <int HD, int NWARPS, int STAGES>
+template <int HD, int NWARPS, int STAGES, bool SIG = false>
 static int launch_flash(const void* q, long long q_row_stride, const void* cache,
                         const int* block_table, int table_stride, const int* cu_q,
                         const int* seqlens_k, void* out, float* part_o, float* part_ml, int num_seqs,
                         int max_q, int nh, int nkv, int page_size, int num_pages, float scale,
                         int window, int splits, int* status, cudaStream_t stream, int q_below = 0, int rows_above = 0,
                         int mask_chunk = 0, const float* sinks = nullptr, const void* gate = nullptr, long long gate_stride = 0,
-                        int keep = 0) {
+                        int keep = 0, const ScoreForm& form = ScoreForm()) {
     const int n_rep = nh / nkv;
     const long long max_rows = (long long)max_q * n_rep;
     const long long tiles = (max_rows + NWARPS * 16 - 1) / (NWARPS * 16);
@@ -346,7 +456,7 @@ static int launch_flash(const void* q, long long q_row_stride, const void* cache
     if (nkv > 65535 || (long long)num_seqs * splits > 65535)
         return fail(-1, "paged_attention: %d kv heads or %d sequences x %d splits exceed the grid", nkv, num_seqs, splits);
     const size_t smem = (size_t)2 * STAGES * FA_BK * HD * sizeof(__nv_bfloat16);
-    auto kern = flash_paged_kernel<HD, NWARPS, STAGES>;
+    auto kern = flash_paged_kernel<HD, NWARPS, STAGES, SIG>;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return fail(-101, "paged_attention: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
@@ -356,7 +466,8 @@ static int launch_flash(const void* q, long long q_row_stride, const void* cache
         (const __nv_bfloat16*)q, q_row_stride, (const __nv_bfloat16*)cache, block_table, table_stride, cu_q,
         seqlens_k, (__nv_bfloat16*)out, part_o, part_ml, nh, nkv, page_size, num_pages,
         scale * 1.4426950408889634f, window, splits, q_below, rows_above, status, mask_chunk, sinks,
-        (const __nv_bfloat16*)gate, gate_stride, keep));
+        (const __nv_bfloat16*)gate, gate_stride, keep, sigmoid_form(scale, form.softcap), form.bias, form.out_scale,
+        form.out_stride));
 }
 
 }  // namespace vapi

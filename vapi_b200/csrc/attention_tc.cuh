@@ -26,10 +26,14 @@
 // their scores are replaced by -inf by selection, and their V rows are zeroed in shared memory
 // before P.V, so that 0 * garbage cannot produce a NaN.
 //
+// A second form of the kernel takes sigmoids of the (capped) scores for weights, without a normalisation over the keys
+// (ScoreForm in attention_mma.cuh): no running maximum, no sums and no rescaling of the accumulator then.
+//
 // Every mbarrier wait is bounded; a role that gives up records status 16 and the block drains
 // (tensor memory is released on every path).
 #pragma once
 #include "tcgen05.cuh"
+#include "attention_mma.cuh"
 
 namespace vapi {
 
@@ -62,6 +66,11 @@ struct FaTcParams {
     const float* sinks;
     const __nv_bfloat16* gate;
     long long gate_stride;
+    // weights that are sigmoids of the scores, not normalised over the keys; bias: a number per head in the score
+    SigmoidForm sig;
+    const float* score_bias;
+    float out_scale;           // the output is multiplied by it
+    long long out_stride;      // elements between two tokens' output rows
 };
 
 __device__ __forceinline__ float ex2_approx(float x) {
@@ -70,6 +79,7 @@ __device__ __forceinline__ float ex2_approx(float x) {
     return y;
 }
 
+template <bool SIG>
 __global__ void __launch_bounds__(FT_THREADS, 2)
 flash_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const FaTcParams p) {
     extern __shared__ unsigned char ft_smem_raw[];
@@ -221,6 +231,7 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const FaTcParams p) {
             mbar_arrive(q_ready);
         }
         float m_run = -INFINITY, l_run = 0.f;
+        const float nb = (SIG && p.score_bias) ? -1.4426950408889634f * p.score_bias[head] : 0.f;
         bool ok = true;
         for (int i = 0; i < nt && ok; ++i) {
             const int sb = i & 1, stage = i % FT_STAGES;
@@ -246,6 +257,9 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const FaTcParams p) {
             const bool need_mask = partial || (k0 + FT_BK - 1 > p_min) || (k0 + FT_BK > klen) ||
                                    (p.window > 0 && k0 <= p_max - p.window) ||
                                    (p.mask_chunk > 0 && k0 < (p_max / p.mask_chunk) * p.mask_chunk);
+            float m_use = 0.f;
+            float rs4[4] = {0.f, 0.f, 0.f, 0.f};
+            if (!SIG) {
             // (four running maxima and, below, four running sums: a single chain of 64 dependent
             // operations would leave the few warps of an SM waiting on latency)
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -280,17 +294,40 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const FaTcParams p) {
                 }
                 tmem_st_wait();
             }
-            // this tile's P buffer was last read by P.V of the tile two before
-            if (i >= 2 && !__all_sync(0xffffffffu, mbar_wait(pv_done + 8 * sb, ((i >> 1) - 1) & 1))) { ok = false; break; }
             l_run *= alpha;
             m_run = m_new;
-            const float m_use = m_run == -INFINITY ? 0.f : m_run;
-            float rs4[4] = {0.f, 0.f, 0.f, 0.f};
+            m_use = m_run == -INFINITY ? 0.f : m_run;
+            } else {
+#pragma unroll
+                for (int c = 0; c < FT_BK / 16; ++c) {
+                    float w16[16];
+#pragma unroll
+                    for (int e = 0; e < 16; ++e) w16[e] = sv[c * 16 + e];
+                    sigmoid_weights(w16, p.sig, nb);
+#pragma unroll
+                    for (int e = 0; e < 16; ++e) sv[c * 16 + e] = w16[e];
+                }
+                if (need_mask) {
+#pragma unroll
+                    for (int e = 0; e < FT_BK; ++e) {
+                        const int kj = k0 + e;
+                        const bool vis = kj <= pos && kj < klen && (p.window <= 0 || kj > pos - p.window || kj < p.keep) && kj >= pos_lo;
+                        sv[e] = vis ? sv[e] : 0.f;
+                    }
+                }
+            }
+            // this tile's P buffer was last read by P.V of the tile two before
+            if (i >= 2 && !__all_sync(0xffffffffu, mbar_wait(pv_done + 8 * sb, ((i >> 1) - 1) & 1))) { ok = false; break; }
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
                 unsigned w[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
+                    if (SIG) {
+                        __nv_bfloat162 h2 = __floats2bfloat162_rn(sv[c * 8 + 2 * e], sv[c * 8 + 2 * e + 1]);
+                        w[e] = *reinterpret_cast<unsigned*>(&h2);
+                        continue;
+                    }
                     const float a = ex2_approx(fmaf(sv[c * 8 + 2 * e], p.scale_log2e, -m_use));
                     const float b = ex2_approx(fmaf(sv[c * 8 + 2 * e + 1], p.scale_log2e, -m_use));
                     rs4[e] += a + b;
@@ -316,10 +353,11 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap tm_kv, const FaTcParams p) {
         if (ok && !__all_sync(0xffffffffu, mbar_wait(pv_done + 8 * ((nt - 1) & 1), ((nt - 1) >> 1) & 1))) ok = false;
         tc5_fence_after();
         if (ok) {                                                   // (uniform over the warp)
-            if (p.sinks && m_run != -INFINITY) l_run += exp2f(p.sinks[head] * 1.4426950408889634f - m_run);
-            float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+            if (!SIG && p.sinks && m_run != -INFINITY) l_run += exp2f(p.sinks[head] * 1.4426950408889634f - m_run);
+            float inv = SIG ? 1.f : (l_run > 0.f ? 1.f / l_run : 0.f);
             if (p.gate) inv *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[(size_t)(q0 + tok) * p.gate_stride + head])));
-            __nv_bfloat16* o = p.out + ((size_t)(q0 + tok) * p.nh + head) * FT_HD;
+            inv *= p.out_scale;
+            __nv_bfloat16* o = p.out + (size_t)(q0 + tok) * p.out_stride + (size_t)head * FT_HD;
 #pragma unroll
             for (int j = 0; j < FT_HD / 16; ++j) {
                 float o16[16];
@@ -365,24 +403,26 @@ static int make_kv_map(CUtensorMap* map, const void* cache, long long rows) {
     return 0;
 }
 
+template <bool SIG = false>
 static int launch_flash_tc(const void* q, long long q_row_stride, const void* cache, const int* block_table,
                            int table_stride, const int* cu_q, const int* seqlens_k, void* out, int num_seqs,
                            int max_q, int nh, int nkv, int page_size, int num_pages, float scale, int window,
                            int min_q, int* status, cudaStream_t stream, int mask_chunk = 0, const float* sinks = nullptr,
-                           const void* gate = nullptr, long long gate_stride = 0, int keep = 0) {
+                           const void* gate = nullptr, long long gate_stride = 0, int keep = 0,
+                           const ScoreForm& form = ScoreForm()) {
     const int n_rep = nh / nkv;
     const long long tiles = ((long long)max_q * n_rep + FT_ROWS - 1) / FT_ROWS;
     if (tiles > 0x7fffffffLL || nkv > 65535 || num_seqs > 65535)
         return fail(-1, "paged_attention: the step exceeds the grid (%lld row tiles, %d kv heads, %d sequences)", tiles, nkv, num_seqs);
     if (!(scale > 0.f)) return fail(-1, "paged_attention: the tcgen05 kernel needs a positive scale");
-    if (q_row_stride % 8 != 0 || ((uintptr_t)q & 15) != 0 || ((uintptr_t)out & 15) != 0)
+    if (q_row_stride % 8 != 0 || ((uintptr_t)q & 15) != 0 || ((uintptr_t)out & 15) != 0 || form.out_stride % 8 != 0)
         return fail(-1, "paged_attention: the tcgen05 kernel needs 16-byte aligned query and output rows");
     CUtensorMap map;
     int rc = make_kv_map(&map, cache, (long long)num_pages * 2 * nkv * page_size);
     if (rc != 0) return rc;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FT_SMEM);
+        cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel<SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FT_SMEM);
         if (e != cudaSuccess) return fail(-101, "paged_attention: cannot reserve %zu bytes of shared memory: %s", FT_SMEM, cudaGetErrorString(e));
         attr_set = true;
     }
@@ -391,8 +431,10 @@ static int launch_flash_tc(const void* q, long long q_row_stride, const void* ca
     p.cu_q = cu_q; p.seqlens_k = seqlens_k; p.out = (__nv_bfloat16*)out; p.nh = nh; p.nkv = nkv; p.page_size = page_size;
     p.num_pages = num_pages; p.scale_log2e = scale * 1.4426950408889634f; p.window = window; p.min_q = min_q; p.status = status;
     p.mask_chunk = mask_chunk; p.keep = keep; p.sinks = sinks; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride;
+    p.sig = sigmoid_form(scale, form.softcap); p.score_bias = form.bias; p.out_scale = form.out_scale;
+    p.out_stride = form.out_stride > 0 ? form.out_stride : (long long)nh * FT_HD;
     dim3 grid((unsigned)tiles, nkv, num_seqs);
-    return check_launch("paged_attention (tcgen05)", launch(flash_tc_kernel, grid, FT_THREADS, FT_SMEM, stream, map, p));
+    return check_launch("paged_attention (tcgen05)", launch(flash_tc_kernel<SIG>, grid, FT_THREADS, FT_SMEM, stream, map, p));
 }
 
 }  // namespace vapi

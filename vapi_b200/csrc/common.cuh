@@ -155,6 +155,14 @@ template <typename T> __device__ __forceinline__ float round_to(float v) {
     return to_f32(from_f32<T>(v));
 }
 
+// ---- an activation that products apply as their epilogue ----------------------------------
+// xIELU: up * z^2 + z / 2 for z > 0, down * (exp(z) - 1 - z) + z / 2 for z <= 0, with two numbers
+// a layer owns (both already positive: the caller passes softplus(p) and 1/2 + softplus(q)).
+__device__ __forceinline__ float xielu(float z, float up, float down) {
+    const float half = 0.5f * z;
+    return z > 0.f ? fmaf(up * z, z, half) : fmaf(down, expm1f(z) - z, half);
+}
+
 // ---- warp / block reductions -----------------------------------------------
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

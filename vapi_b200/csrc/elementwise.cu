@@ -88,6 +88,84 @@ VAPI_EXPORT int vapi_resolve_tokens(int* tokens, const int* src, const int* prev
 }
 
 // ---------------------------------------------------------------------------
+// embedding with a bigram row added:  out[t] = float(table[token]) * scale + float(bigram[row]), where
+//   row = (previous token * mul_prev + token * mul_cur) mod buckets,  and the last row, number `buckets`, for the
+// first token of a sequence.  The previous token of a sequence's first token of the step comes from the request's
+// state slot (one int), and the block that reads it there also stores the sequence's last token of the step: nobody
+// else touches the slot, so nothing is read after it was replaced.  Slots are never cleared: position 0 says that
+// there is no previous token.
+template <typename TW>
+__global__ void embed_bigram_kernel(const TW* __restrict__ table, const TW* __restrict__ bigram,
+                                    const int* __restrict__ tokens, const int* __restrict__ positions,
+                                    const int* __restrict__ tok_seq, const int* __restrict__ cu_q,
+                                    const int* __restrict__ state_slots, int* __restrict__ state, long long slot_stride,
+                                    int num_slots, long long mul_prev, long long mul_cur, int buckets,
+                                    float* __restrict__ out, int n, int hidden, int vocab, float scale,
+                                    int* __restrict__ status) {
+    __shared__ int row_sh;
+    const int t = blockIdx.x;
+    pdl_trigger();
+    pdl_wait();
+    if (t >= n) return;
+    int tok = tokens[t];
+    if (tok < 0 || tok >= vocab) {  // never read outside the table
+        if (threadIdx.x == 0 && status) atomicExch(status, 1);
+        tok = 0;
+    }
+    if (threadIdx.x == 0) {
+        const int seq = tok_seq[t], first = cu_q[seq];
+        int prev = -1;
+        if (t > first) {
+            prev = tokens[t - 1];
+        } else {
+            const int slot = state_slots[seq];
+            if (slot < 0 || slot >= num_slots) {
+                if (status) atomicExch(status, 3);
+            } else {
+                int* st = state + (size_t)slot * slot_stride;
+                if (positions[t] > 0) prev = *st;
+                *st = tokens[cu_q[seq + 1] - 1];
+            }
+        }
+        int row = buckets;
+        if (prev >= 0) {
+            long long v = ((long long)prev * mul_prev + (long long)tok * mul_cur) % buckets;
+            row = (int)(v < 0 ? v + buckets : v);
+        }
+        row_sh = row;
+    }
+    __syncthreads();
+    const TW* src = table + (size_t)tok * hidden;
+    const TW* add = bigram + (size_t)row_sh * hidden;
+    float* dst = out + (size_t)t * hidden;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = fmaf(to_f32(src[c]), scale, to_f32(add[c]));
+}
+
+VAPI_EXPORT int vapi_embed_bigram(const void* table, const void* bigram, int table_dtype, const int* tokens,
+                                  const int* positions, const int* tok_seq, const int* cu_q, const int* state_slots,
+                                  int* state, long long slot_stride, int num_slots, long long mul_prev, long long mul_cur,
+                                  int buckets, float* out, int n, int hidden, int vocab, float scale, int* status,
+                                  cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (hidden <= 0 || vocab <= 0 || buckets <= 0 || num_slots <= 0)
+        return fail(-1, "embed_bigram: hidden=%d vocab=%d buckets=%d slots=%d", hidden, vocab, buckets, num_slots);
+    if (!table || !bigram || !state || !state_slots || !tok_seq || !cu_q || !positions) return fail(-1, "embed_bigram: missing array");
+    const int threads = hidden >= 1024 ? 256 : 128;
+    cudaError_t e;
+    if (table_dtype == VAPI_F32)
+        e = launch(embed_bigram_kernel<float>, n, threads, 0, stream, (const float*)table, (const float*)bigram, tokens, positions,
+                   tok_seq, cu_q, state_slots, state, slot_stride, num_slots, mul_prev, mul_cur, buckets, out, n, hidden, vocab,
+                   scale, status);
+    else if (table_dtype == VAPI_BF16)
+        e = launch(embed_bigram_kernel<__nv_bfloat16>, n, threads, 0, stream, (const __nv_bfloat16*)table,
+                   (const __nv_bfloat16*)bigram, tokens, positions, tok_seq, cu_q, state_slots, state, slot_stride, num_slots,
+                   mul_prev, mul_cur, buckets, out, n, hidden, vocab, scale, status);
+    else
+        return fail(-2, "embed_bigram: unsupported table dtype %d", table_dtype);
+    return check_launch("embed_bigram", e);
+}
+
+// ---------------------------------------------------------------------------
 // fused residual add + RMSNorm.
 //   if delta: x[row] += float(delta[row])           (x is the float residual stream)
 //   out[j]   = T( x[row] * rsqrt(mean(x[row]^2) + eps) * w )
@@ -356,6 +434,207 @@ VAPI_EXPORT int vapi_scaled_add_rmsnorm(float* x, const void* y1, const float* s
     else return fail(-2, "scaled_add_rmsnorm: unsupported dtype %d", dtype);
 #undef SAR_GO
     return check_launch("scaled_add_rmsnorm", e);
+}
+
+// The pending outputs of two sublayers folded into the stream, the norm, and a token shift behind it, in one pass:
+//   v_t = x_t + s1 * y1_t + s2 * y2_t  (y2 or both may be absent; a scale may be absent and then counts as one)
+//   h_t = rmsnorm(v_t) * w
+//   out_h[t] = T(h_t),   out_s[t] = T(h_t + (h_{t-1} - h_t) * shift)
+// h_{t-1} is the previous token of the same sequence, zeros before position 0.  It is worked out again from row t - 1
+// of the inputs (same threads, same order of additions, hence the same bits), so no block waits for another; that is
+// why the new stream goes to x_out and not back into x (x_out may be null when nothing is pending: x is then the
+// stream already).  A sequence's first token of the step takes h_{t-1} from the request's state slot (float [hidden]),
+// and the same threads then store the h of the sequence's last token of the step there: nobody else touches the slot.
+// A block takes `rows_per_block` tokens one after another and hands h on in registers.
+struct ShiftIndex {
+    const int* positions; const int* tok_seq; const int* cu_q; const int* state_slots;
+    float* state; long long slot_stride; int num_slots; int* status;
+};
+
+constexpr int SHIFT_KMAX = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+shift_add_rmsnorm_vec_kernel(const float* __restrict__ x, const T* __restrict__ y1, const float* __restrict__ s1,
+                             const T* __restrict__ y2, const float* __restrict__ s2, const float* __restrict__ w, float eps,
+                             const float* __restrict__ shift, const ShiftIndex ix, float* __restrict__ x_out,
+                             T* __restrict__ out_h, T* __restrict__ out_s, int n, int hidden, int rows_per_block) {
+    __shared__ float red[33];
+    const int h4 = hidden >> 2;
+    const int t0 = blockIdx.x * rows_per_block, t1 = min(n, t0 + rows_per_block);
+    pdl_trigger();
+    pdl_wait();
+    // h of a row; with `keep` its stream is stored
+    auto norm_row = [&](int t, float4 (&v)[SHIFT_KMAX], bool keep) {
+        const float* xr = x + (size_t)t * hidden;
+        const T* a = y1 ? y1 + (size_t)t * hidden : nullptr;
+        const T* b = y2 ? y2 + (size_t)t * hidden : nullptr;
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < SHIFT_KMAX; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (c < h4) {
+                v[k] = Pack4<float>::load(xr + 4 * c);
+                if (a) {
+                    const float4 d = Pack4<T>::load(a + 4 * c);
+                    const float4 s = s1 ? Pack4<float>::load(s1 + 4 * c) : make_float4(1.f, 1.f, 1.f, 1.f);
+                    v[k].x += s.x * d.x; v[k].y += s.y * d.y; v[k].z += s.z * d.z; v[k].w += s.w * d.w;
+                }
+                if (b) {
+                    const float4 d = Pack4<T>::load(b + 4 * c);
+                    const float4 s = s2 ? Pack4<float>::load(s2 + 4 * c) : make_float4(1.f, 1.f, 1.f, 1.f);
+                    v[k].x += s.x * d.x; v[k].y += s.y * d.y; v[k].z += s.z * d.z; v[k].w += s.w * d.w;
+                }
+                if (keep && x_out) Pack4<float>::store(x_out + (size_t)t * hidden + 4 * c, v[k]);
+                ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+            }
+        }
+        ss = block_sum(ss, red);
+        const float inv = rsqrtf(ss / (float)hidden + eps);
+#pragma unroll
+        for (int k = 0; k < SHIFT_KMAX; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < h4) {
+                const float4 wv = Pack4<float>::load(w + 4 * c);
+                v[k].x *= inv * wv.x; v[k].y *= inv * wv.y; v[k].z *= inv * wv.z; v[k].w *= inv * wv.w;
+            }
+        }
+    };
+    float4 prev[SHIFT_KMAX], cur[SHIFT_KMAX];
+#pragma unroll
+    for (int k = 0; k < SHIFT_KMAX; ++k) prev[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int t = t0; t < t1; ++t) {
+        const int seq = ix.tok_seq[t];
+        const bool first = t == ix.cu_q[seq];
+        float* st = nullptr;
+        if (first) {
+            const int slot = ix.state_slots[seq];
+            if (slot < 0 || slot >= ix.num_slots) {
+                if (threadIdx.x == 0 && ix.status) atomicExch(ix.status, 3);
+            } else {
+                st = ix.state + (size_t)slot * ix.slot_stride;
+            }
+            const bool carry = st && ix.positions[t] > 0;
+#pragma unroll
+            for (int k = 0; k < SHIFT_KMAX; ++k) {
+                const int c = threadIdx.x + k * blockDim.x;
+                prev[k] = (carry && c < h4) ? Pack4<float>::load(st + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        } else if (t == t0) {
+            norm_row(t - 1, prev, false);
+        }
+        norm_row(t, cur, true);
+#pragma unroll
+        for (int k = 0; k < SHIFT_KMAX; ++k) {
+            const int c = threadIdx.x + k * blockDim.x;
+            if (c < h4) {
+                const float4 m = Pack4<float>::load(shift + 4 * c);
+                const float4 h = cur[k], p = prev[k];
+                if (out_h) Pack4<T>::store(out_h + (size_t)t * hidden + 4 * c, h);
+                Pack4<T>::store(out_s + (size_t)t * hidden + 4 * c,
+                                make_float4(fmaf(p.x - h.x, m.x, h.x), fmaf(p.y - h.y, m.y, h.y), fmaf(p.z - h.z, m.z, h.z),
+                                            fmaf(p.w - h.w, m.w, h.w)));
+            }
+        }
+        if (st) {
+            const int last = ix.cu_q[seq + 1] - 1;
+            if (last != t) norm_row(last, prev, false);
+#pragma unroll
+            for (int k = 0; k < SHIFT_KMAX; ++k) {
+                const int c = threadIdx.x + k * blockDim.x;
+                if (c < h4) Pack4<float>::store(st + 4 * c, last != t ? prev[k] : cur[k]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < SHIFT_KMAX; ++k) prev[k] = cur[k];
+    }
+}
+
+// Any width: a block a token, elements one by one, the previous row's h worked out again where it is needed.
+template <typename T>
+__global__ void shift_add_rmsnorm_kernel(const float* __restrict__ x, const T* __restrict__ y1, const float* __restrict__ s1,
+                                         const T* __restrict__ y2, const float* __restrict__ s2, const float* __restrict__ w,
+                                         float eps, const float* __restrict__ shift, const ShiftIndex ix,
+                                         float* __restrict__ x_out, T* __restrict__ out_h, T* __restrict__ out_s, int n,
+                                         int hidden) {
+    __shared__ float red[33];
+    const int t = blockIdx.x;
+    pdl_trigger();
+    pdl_wait();
+    if (t >= n) return;
+    auto value = [&](int r, int c) {
+        const size_t i = (size_t)r * hidden + c;
+        float v = x[i];
+        if (y1) v += (s1 ? s1[c] : 1.f) * to_f32(y1[i]);
+        if (y2) v += (s2 ? s2[c] : 1.f) * to_f32(y2[i]);
+        return v;
+    };
+    auto inverse = [&](int r) {
+        float ss = 0.f;
+        for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+            const float v = value(r, c);
+            ss += v * v;
+        }
+        return rsqrtf(block_sum(ss, red) / (float)hidden + eps);
+    };
+    const int seq = ix.tok_seq[t];
+    const bool first = t == ix.cu_q[seq];
+    const int last = ix.cu_q[seq + 1] - 1;
+    float* st = nullptr;
+    if (first) {
+        const int slot = ix.state_slots[seq];
+        if (slot < 0 || slot >= ix.num_slots) {
+            if (threadIdx.x == 0 && ix.status) atomicExch(ix.status, 3);
+        } else {
+            st = ix.state + (size_t)slot * ix.slot_stride;
+        }
+    }
+    const bool carry = st && ix.positions[t] > 0;
+    const float inv = inverse(t);
+    const float inv_prev = first ? 0.f : inverse(t - 1);
+    const float inv_last = (first && last != t) ? inverse(last) : inv;
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+        const float v = value(t, c);
+        const float h = v * (inv * w[c]);
+        const float p = first ? (carry ? st[c] : 0.f) : value(t - 1, c) * (inv_prev * w[c]);
+        if (x_out) x_out[(size_t)t * hidden + c] = v;
+        if (out_h) out_h[(size_t)t * hidden + c] = from_f32<T>(h);
+        out_s[(size_t)t * hidden + c] = from_f32<T>(fmaf(p - h, shift[c], h));
+        if (st) st[c] = last == t ? h : value(last, c) * (inv_last * w[c]);
+    }
+}
+
+VAPI_EXPORT int vapi_shift_add_rmsnorm(const float* x, const void* y1, const float* s1, const void* y2, const float* s2,
+                                       const float* w, float eps, const float* shift, const int* positions,
+                                       const int* tok_seq, const int* cu_q, const int* state_slots, float* state,
+                                       long long slot_stride, int num_slots, float* x_out, void* out_h, void* out_s, int dtype,
+                                       int n, int hidden, int rows_per_block, int* status, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (hidden <= 0 || num_slots <= 0 || slot_stride < 0) return fail(-1, "shift_add_rmsnorm: hidden=%d, %d slots", hidden, num_slots);
+    if (!y1 && y2) return fail(-1, "shift_add_rmsnorm: the second sublayer comes with a first");
+    if (y1 && (!x_out || x_out == x)) return fail(-1, "shift_add_rmsnorm: with something pending the new stream needs memory of its own");
+    if (!w || !shift || !state || !out_s || !positions || !tok_seq || !cu_q || !state_slots)
+        return fail(-1, "shift_add_rmsnorm: missing array");
+    ShiftIndex ix = {positions, tok_seq, cu_q, state_slots, state, slot_stride, num_slots, status};
+    const int esz = dtype == VAPI_F32 ? 4 : 2;
+    const bool aligned = (((uintptr_t)x | (uintptr_t)x_out | (uintptr_t)s1 | (uintptr_t)s2 | (uintptr_t)w | (uintptr_t)shift |
+                           (uintptr_t)state) & 15) == 0 && slot_stride % 4 == 0 &&
+                         (((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)out_h | (uintptr_t)out_s) & (4 * esz - 1)) == 0;
+    const int vt = hidden > 1024 ? 256 : 128;
+    const bool vec = hidden % 4 == 0 && hidden / 4 <= SHIFT_KMAX * vt && aligned;
+    const int rpb = rows_per_block > 0 ? rows_per_block : 1;
+    cudaError_t e;
+#define SHIFT_GO(T)                                                                                                            \
+    e = vec ? launch(shift_add_rmsnorm_vec_kernel<T>, (n + rpb - 1) / rpb, vt, 0, stream, x, (const T*)y1, s1, (const T*)y2,   \
+                     s2, w, eps, shift, ix, x_out, (T*)out_h, (T*)out_s, n, hidden, rpb)                                       \
+            : launch(shift_add_rmsnorm_kernel<T>, n, 256, 0, stream, x, (const T*)y1, s1, (const T*)y2, s2, w, eps, shift, ix, \
+                     x_out, (T*)out_h, (T*)out_s, n, hidden)
+    if (dtype == VAPI_F32) SHIFT_GO(float);
+    else if (dtype == VAPI_BF16) SHIFT_GO(__nv_bfloat16);
+    else return fail(-2, "shift_add_rmsnorm: unsupported dtype %d", dtype);
+#undef SHIFT_GO
+    return check_launch("shift_add_rmsnorm", e);
 }
 
 // residual add alone (used at the very end of a step when nothing follows the
@@ -727,9 +1006,45 @@ VAPI_EXPORT int vapi_postnorm_add_rmsnorm(float* x, const void* y, int dtype, co
     return check_launch("postnorm_add_rmsnorm", e);
 }
 
+// xIELU elementwise (where it does not ride on a product): out = xielu(z), consts = {up, down}; four elements a
+// thread with 8- / 16-byte accesses, the last few one by one.
+template <typename T>
+__global__ void xielu_kernel(const T* __restrict__ z, T* __restrict__ out, const float* __restrict__ consts, size_t total, int vec) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    pdl_trigger();
+    pdl_wait();
+    const float up = consts[0], down = consts[1];
+    const size_t i0 = i * 4;
+    if (vec && i0 + 3 < total) {
+        const float4 v = Pack4<T>::load(z + i0);
+        Pack4<T>::store(out + i0, make_float4(xielu(v.x, up, down), xielu(v.y, up, down), xielu(v.z, up, down), xielu(v.w, up, down)));
+    } else {
+        for (size_t j = i0; j < i0 + 4 && j < total; ++j) out[j] = from_f32<T>(xielu(to_f32(z[j]), up, down));
+    }
+}
+
+VAPI_EXPORT int vapi_xielu(const void* z, void* out, int dtype, const float* consts, long long total, cudaStream_t stream) {
+    if (total <= 0) return 0;
+    if (!consts) return fail(-1, "xielu: the activation's two numbers are missing");
+    const int esz = dtype == VAPI_F32 ? 4 : 2;
+    const int vec = (((uintptr_t)z | (uintptr_t)out) & (4 * esz - 1)) == 0;
+    const long long blocks = ((total + 3) / 4 + 255) / 256;
+    if (blocks > 0x7fffffffLL) return fail(-1, "xielu: %lld elements", total);
+    cudaError_t e;
+    if (dtype == VAPI_F32)
+        e = launch(xielu_kernel<float>, (int)blocks, 256, 0, stream, (const float*)z, (float*)out, consts, (size_t)total, vec);
+    else if (dtype == VAPI_BF16)
+        e = launch(xielu_kernel<__nv_bfloat16>, (int)blocks, 256, 0, stream, (const __nv_bfloat16*)z, (__nv_bfloat16*)out, consts,
+                   (size_t)total, vec);
+    else
+        return fail(-2, "xielu: unsupported dtype %d", dtype);
+    return check_launch("xielu", e);
+}
+
 // RMS norm over equal groups of a row, with a gate:  out = norm_g(y) * w * silu(z)  (gate_first 0)
 // or  out = norm_g(y * silu(z)) * w  (gate_first 1).  y is float [n, width] (what a recurrence
-// left), z is T with its own row stride, w has w_len elements and is indexed by column % w_len (one
+// left), z is T with its own row stride, out has rows of `out_stride` elements (it may be the right part of a wider
+// buffer), w has w_len elements and is indexed by column % w_len (one
 // weight per head size, or one per column).  `gate_first` carries two bits: bit 0 the order above, bit 1 the
 // gate's kind (0: silu(z), 2: sigmoid(z)).  One warp per (row, group).
 __device__ __forceinline__ float norm_gate(float zv, int sigmoid_gate) {
@@ -739,7 +1054,7 @@ __device__ __forceinline__ float norm_gate(float zv, int sigmoid_gate) {
 template <typename T>
 __global__ void gated_group_rmsnorm_kernel(const float* __restrict__ y, const T* __restrict__ z, long long z_stride,
                                            const float* __restrict__ w, int w_len, float eps, int gate_first,
-                                           T* __restrict__ out, int n, int width, int group) {
+                                           T* __restrict__ out, int n, int width, int group, long long out_stride) {
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     pdl_trigger();
@@ -762,7 +1077,7 @@ __global__ void gated_group_rmsnorm_kernel(const float* __restrict__ y, const T*
     }
     ss = warp_sum(ss);
     const float inv = rsqrtf(ss / (float)group + eps);
-    T* orow = out + (size_t)t * width + (size_t)g * group;
+    T* orow = out + (size_t)t * out_stride + (size_t)g * group;
     for (int c = lane; c < group; c += 32) {
         const float zv = to_f32(zr[c]);
         const float gate = norm_gate(zv, sig);
@@ -776,7 +1091,7 @@ __global__ void gated_group_rmsnorm_kernel(const float* __restrict__ y, const T*
 template <typename T>
 __global__ void gated_group_rmsnorm_wide_kernel(const float* __restrict__ y, const T* __restrict__ z, long long z_stride,
                                                 const float* __restrict__ w, int w_len, float eps, int gate_first,
-                                                T* __restrict__ out, int n, int width, int group) {
+                                                T* __restrict__ out, int n, int width, int group, long long out_stride) {
     __shared__ float red[33];
     const int groups = width / group;
     const int t = blockIdx.x / groups, g = blockIdx.x - t * groups;
@@ -797,7 +1112,7 @@ __global__ void gated_group_rmsnorm_wide_kernel(const float* __restrict__ y, con
     }
     ss = block_sum(ss, red);
     const float inv = rsqrtf(ss / (float)group + eps);
-    T* orow = out + (size_t)t * width + (size_t)g * group;
+    T* orow = out + (size_t)t * out_stride + (size_t)g * group;
     for (int c = threadIdx.x; c < group; c += blockDim.x) {
         const float zv = to_f32(zr[c]);
         const float gate = norm_gate(zv, sig);
@@ -808,8 +1123,9 @@ __global__ void gated_group_rmsnorm_wide_kernel(const float* __restrict__ y, con
 
 VAPI_EXPORT int vapi_gated_group_rmsnorm(const float* y, const void* z, long long z_stride, int dtype, const float* w,
                                          int w_len, float eps, int gate_first, void* out, int n, int width, int group,
-                                         cudaStream_t stream) {
+                                         cudaStream_t stream, long long out_stride) {
     if (n <= 0) return 0;
+    if (out_stride < width) return fail(-1, "gated_group_rmsnorm: output rows of %lld elements for a width of %d", out_stride, width);
     if (width <= 0 || group <= 0 || width % group || w_len <= 0)
         return fail(-1, "gated_group_rmsnorm: width %d, group %d, weight %d", width, group, w_len);
     const long long items = (long long)n * (width / group);
@@ -820,18 +1136,18 @@ VAPI_EXPORT int vapi_gated_group_rmsnorm(const float* y, const void* z, long lon
         const int threads = group >= 2048 ? 256 : 128;
         if (dtype == VAPI_F32)
             e = launch(gated_group_rmsnorm_wide_kernel<float>, (int)items, threads, 0, stream, y, (const float*)z, z_stride, w,
-                       w_len, eps, gate_first, (float*)out, n, width, group);
+                       w_len, eps, gate_first, (float*)out, n, width, group, out_stride);
         else
             e = launch(gated_group_rmsnorm_wide_kernel<__nv_bfloat16>, (int)items, threads, 0, stream, y, (const __nv_bfloat16*)z,
-                       z_stride, w, w_len, eps, gate_first, (__nv_bfloat16*)out, n, width, group);
+                       z_stride, w, w_len, eps, gate_first, (__nv_bfloat16*)out, n, width, group, out_stride);
         return check_launch("gated_group_rmsnorm", e);
     }
     if (dtype == VAPI_F32)
         e = launch(gated_group_rmsnorm_kernel<float>, blocks, warps * 32, 0, stream, y, (const float*)z, z_stride, w, w_len, eps,
-                   gate_first, (float*)out, n, width, group);
+                   gate_first, (float*)out, n, width, group, out_stride);
     else if (dtype == VAPI_BF16)
         e = launch(gated_group_rmsnorm_kernel<__nv_bfloat16>, blocks, warps * 32, 0, stream, y, (const __nv_bfloat16*)z, z_stride,
-                   w, w_len, eps, gate_first, (__nv_bfloat16*)out, n, width, group);
+                   w, w_len, eps, gate_first, (__nv_bfloat16*)out, n, width, group, out_stride);
     else
         return fail(-2, "gated_group_rmsnorm: unsupported dtype %d", dtype);
     return check_launch("gated_group_rmsnorm", e);

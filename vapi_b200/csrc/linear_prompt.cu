@@ -60,6 +60,7 @@ struct PlParams {
     __nv_bfloat16* out_bf16; float* out_f32; long long out_stride;
     const float* bias; float* resid; float* ss_out; const float* next_w; __nv_bfloat16* xw_out;
     int* status;
+    const float* xielu;                            // EPI_BF16: null, or {up, down}: the output passes xIELU
 };
 
 template <int BN, int PAIR> struct PlCfg {
@@ -365,6 +366,11 @@ prompt_linear_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
                     float v[32];
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) * scale + colv[c + j];
+                    if (p.xielu) {
+                        const float up = p.xielu[0], down = p.xielu[1];
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) v[j] = xielu(v[j], up, down);
+                    }
                     if (fast) {
                         put(v);
                         __syncwarp();
@@ -565,8 +571,9 @@ VAPI_EXPORT int vapi_prompt_linear(const void* W, int N, int K, int M, int pro, 
                                    const float* ss_in, int ss_parts, float eps, int epi, void* out_bf16,
                                    float* out_f32, long long out_stride, const float* bias, float* resid,
                                    float* ss_out, const float* next_w, void* xw_out, int* status,
-                                   cudaStream_t stream) {
+                                   cudaStream_t stream, const float* xielu_consts) {
     if (M <= 0) return 0;
+    if (xielu_consts && epi != PL_EPI_BF16) return fail(-1, "prompt_linear: xIELU comes with the bfloat16 output");
     if (N <= 0 || K <= 0 || K % 8 != 0) return fail(-1, "prompt_linear: K=%d must be a positive multiple of 8 (N=%d)", K, N);
     if (epi == PL_EPI_SWIGLU && N % 2 != 0) return fail(-1, "prompt_linear: SwiGLU needs an even N");
     if (!tokens) return fail(-1, "prompt_linear: no token operand");
@@ -588,7 +595,7 @@ VAPI_EXPORT int vapi_prompt_linear(const void* W, int N, int K, int M, int pro, 
     p.ss_in = ss_in; p.ss_parts = ss_parts; p.eps = eps;
     p.out_bf16 = (__nv_bfloat16*)out_bf16; p.out_f32 = out_f32; p.out_stride = out_stride; p.bias = bias;
     p.resid = resid; p.ss_out = ss_out; p.next_w = next_w; p.xw_out = (__nv_bfloat16*)xw_out;
-    p.status = status;
+    p.status = status; p.xielu = xielu_consts;
     const bool half_rows = epi == PL_EPI_SWIGLU || pair == 2;      // boxes of BN/2 weight rows
     const CUtensorMap *ta, *tw;
     int rc = pl_map(&ta, tokens, M, K, PL_BM);

@@ -45,6 +45,7 @@ struct TcParams {
     __nv_bfloat16* out_bf16; float* out_f32; long long out_stride;
     const float* bias; float* resid; float* ss_out; const float* next_w; __nv_bfloat16* xw_out;
     int* status;
+    const float* xielu;                                            // EPI_BF16: null, or {up, down}: the output passes xIELU
 };
 
 template <int BN> struct TcCfg {
@@ -198,9 +199,14 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant
         }
         const long long f0 = (long long)n0 + 4 * lane;             // four features per lane
         const float4 v = *reinterpret_cast<const float4*>(f + 4 * lane);
-        const float vv[4] = {v.x, v.y, v.z, v.w};
+        float vv[4] = {v.x, v.y, v.z, v.w};
         const bool full = f0 + 3 < p.N;
         if (p.epi == TC_EPI_BF16) {
+            if (p.xielu) {
+                const float up = p.xielu[0], down = p.xielu[1];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) vv[i] = xielu(vv[i], up, down);
+            }
             __nv_bfloat16* o = p.out_bf16 + (size_t)m * p.out_stride + f0;
             if (full && (p.out_stride & 3) == 0) {
                 uint2 pk;
@@ -399,8 +405,9 @@ VAPI_EXPORT int vapi_linear_tc(const void* W, int N, int K, int M, int pro, cons
                                const float* ss_in, int ss_parts, float eps, int epi, void* out_bf16,
                                float* out_f32, long long out_stride, const float* bias, float* resid,
                                float* ss_out, const float* next_w, void* xw_out, int* status,
-                               cudaStream_t stream) {
+                               cudaStream_t stream, const float* xielu_consts) {
     if (M <= 0) return 0;
+    if (xielu_consts && epi != TC_EPI_BF16) return fail(-1, "linear_tc: xIELU comes with the bfloat16 output");
     if (M > 256) return fail(-1, "linear_tc: %d rows are more than 256", M);
     if (N <= 0 || K <= 0 || K % 8 != 0) return fail(-1, "linear_tc: K=%d must be a positive multiple of 8 (N=%d)", K, N);
     if (epi == TC_EPI_SWIGLU && N % 2 != 0) return fail(-1, "linear_tc: SwiGLU needs an even N");
@@ -418,7 +425,7 @@ VAPI_EXPORT int vapi_linear_tc(const void* W, int N, int K, int M, int pro, cons
     p.ss_in = ss_in; p.ss_parts = ss_parts; p.eps = eps;
     p.out_bf16 = (__nv_bfloat16*)out_bf16; p.out_f32 = out_f32; p.out_stride = out_stride; p.bias = bias;
     p.resid = resid; p.ss_out = ss_out; p.next_w = next_w; p.xw_out = (__nv_bfloat16*)xw_out;
-    p.status = status;
+    p.status = status; p.xielu = xielu_consts;
     CUtensorMap tw, ta;
     int rc = make_map(&tw, W, N, K, epi == TC_EPI_SWIGLU ? 64 : TC_BM);
     if (rc) return rc;

@@ -91,6 +91,11 @@ class ModelRunner:
             else:
                 self._site_of.append(owner if self.cache.site_tensor(owner) is not None else None)
         flat = [s for e in self._site_of for s in (e if isinstance(e, list) else [e]) if s is not None]
+        # what blocks and the embedding keep for themselves, beside their mixers' caches
+        self._block_site = [("block", i) if self.cache.site_tensor(("block", i)) is not None else None
+                            for i in range(len(plan.order))]
+        self._embedding_view = CacheView("state", self.cache.site_tensor("embedding"), spec=self.cache.site_spec("embedding")) \
+            if self.cache.site_tensor("embedding") is not None else None
         self._site_buffers = {s: self.cache.site_buffers(s) for s in set(flat)}
         #: whether every block has the stream form that steps of few rows run (blocks without it hand
         #: their output on in another shape than a plain delta, so such a model takes the ordinary path)
@@ -139,7 +144,7 @@ class ModelRunner:
                 k = 1
                 for d in s.shape:
                     k *= d
-                per_req += k * esize
+                per_req += k * (s.dtype.itemsize if s.dtype is not None else esize)
         if self.device.type != "cuda":
             raise ValueError("num_pages must be given when the device is not CUDA")
         free, _ = torch.cuda.mem_get_info(self.device)
@@ -169,6 +174,8 @@ class ModelRunner:
                 out.append(CacheView("multi", write=write, parts=[one(s, write) for s in site]))
             else:
                 out.append(one(site, write))
+            if self._block_site[i] is not None:
+                out[-1].block = one(self._block_site[i], True)
         return out
 
     def forward(self, ctx: StepContext) -> Optional[torch.Tensor]:
@@ -191,7 +198,7 @@ class ModelRunner:
                           or 0 < ops.PROMPT_MIN_ROWS <= ctx.n))
         if ctx.fused:
             return self._forward_few_rows(ctx, views)
-        x = plan.embedding.forward(ctx)
+        x = self._embed(ctx)
         if plan.stream_parts:
             ctx.extras.clear()          # what a stream part kept belongs to one run of the step (a captured step runs thrice)
         if self._keep_embedding:
@@ -201,11 +208,18 @@ class ModelRunner:
         for i, call in enumerate(plan.order):
             if call.before is not None:
                 x, delta = plan.stream_parts[call.before].forward(x, delta, ctx)
-            delta = plan.layers[call.layer].forward(x, delta, ctx, views[i])
+            out = plan.layers[call.layer].forward(x, delta, ctx, views[i])
+            # (a block may put the new stream into memory of its own)
+            x, delta = out if getattr(plan.layers[call.layer], "replaces_stream", False) else (x, out)
         if ctx.logits_rows is None:
             return None
         xn = plan.final_norm.apply(x, delta, ctx.dtype, rows=ctx.logits_rows)
         return plan.head.forward(xn)
+
+    def _embed(self, ctx: StepContext) -> torch.Tensor:
+        if self._embedding_view is not None:
+            return self.plan.embedding.forward(ctx, cache=self._embedding_view)
+        return self.plan.embedding.forward(ctx)
 
     def _forward_few_rows(self, ctx: StepContext, views: List[CacheView]) -> Optional[torch.Tensor]:
         """The same model for a step of at most 16 rows (decode): every block runs in its

@@ -95,9 +95,16 @@ class ModelPlan:
     def cache_sites(self) -> List[Tuple[object, object]]:
         """(site, spec) of every cache that a call site owns.  A site is the call site's index in the run
         order, or ``(index, member)`` for each member of a mixer that is several mixers side by side (its
-        ``cache_spec`` is a tuple)."""
+        ``cache_spec`` is a tuple); what a block keeps for itself is ``("block", index)``, whoever owns its mixer's
+        cache, and what the embedding keeps ``"embedding"``."""
         out = []
+        spec = self.embedding.block_cache_spec()
+        if spec is not None:
+            out.append(("embedding", spec))
         for i, c in enumerate(self.order):
+            spec = self.layers[c.layer].block_cache_spec()
+            if spec is not None:
+                out.append((("block", i), spec))
             if c.cache_of is None:
                 spec = self.layers[c.layer].mixer.cache_spec()
                 if isinstance(spec, tuple):

@@ -199,6 +199,33 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, status: Optional[torch.Tens
     return (out, ss, xw) if next_weight is not None else out
 
 
+def embed_bigram(table: torch.Tensor, bigram: torch.Tensor, tokens: torch.Tensor, positions: torch.Tensor,
+                 tok_seq: torch.Tensor, cu_q: torch.Tensor, state: torch.Tensor, state_slots: torch.Tensor, mul_prev: int,
+                 mul_cur: int, scale: float = 1.0, status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """:func:`embed` with a row of a second table added: ``table[token] * scale + bigram[row]`` where ``row`` is
+    ``(previous token * mul_prev + token * mul_cur) mod buckets`` and, for the first token of a sequence, ``buckets``
+    (``bigram`` is [buckets + 1, H]).  ``state`` [slots, 1] int32 carries each request's last token from step to step
+    and is moved on."""
+    _cuda(table, bigram, tokens, positions, tok_seq, cu_q, state, state_slots)
+    _contig(table, "embedding table")
+    _contig(bigram, "bigram table")
+    for t, w in ((tokens, "tokens"), (positions, "positions"), (tok_seq, "tok_seq"), (cu_q, "cu_q"), (state_slots, "state slots"),
+                 (state, "previous tokens")):
+        _i32(t, w)
+    n, (vocab, hidden) = tokens.numel(), table.shape
+    if bigram.dtype != table.dtype or bigram.dim() != 2 or bigram.shape[1] != hidden or bigram.shape[0] < 2:
+        raise KernelError("the bigram table must be [buckets + 1, H] of the embedding table's dtype")
+    if state.dim() != 2 or state.shape[1] != 1:
+        raise KernelError("the previous tokens must be [slots, 1]")
+    out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
+    lib = _lib("elementwise")
+    _check(lib, lib.vapi_embed_bigram(
+        _p(table), _p(bigram), _dt(table), _p(tokens), _p(positions), _p(tok_seq), _p(cu_q), _p(state_slots), _p(state),
+        ctypes.c_longlong(state.stride(0)), state.shape[0], ctypes.c_longlong(int(mul_prev)), ctypes.c_longlong(int(mul_cur)),
+        bigram.shape[0] - 1, _p(out), n, hidden, vocab, ctypes.c_float(scale), _p(status), _stream()))
+    return out
+
+
 def add_residual_ss(x: torch.Tensor, delta: torch.Tensor, next_weight: torch.Tensor):
     """``x += delta`` on the float32 stream; returns ``(ss, xw)`` for the norm that follows:
     the sums of squares of the new rows, [1, n], and bfloat16(new row * next_weight)."""
@@ -309,7 +336,7 @@ def skinny_linear(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None,
                   xw: Optional[torch.Tensor] = None, ss_in: Optional[torch.Tensor] = None, eps: float = 0.0,
                   epilogue: str = "bf16", bias: Optional[torch.Tensor] = None,
                   resid: Optional[torch.Tensor] = None, next_weight: Optional[torch.Tensor] = None,
-                  rows_per_block: Optional[int] = None):
+                  rows_per_block: Optional[int] = None, xielu: Optional[torch.Tensor] = None):
     """The weight-streaming product for decode steps (at most 16 rows), with its fusions.
 
     Token operand: ``act`` [M, K] bfloat16; or the residual stream seen through an RMSNorm not
@@ -318,9 +345,11 @@ def skinny_linear(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None,
     norm's ``eps``.  ``epilogue``: "bf16" -> [M, N] bfloat16; "f32" -> [M, N] float32; "swiglu" ->
     [M, N/2] bfloat16 = silu(first half) * second half; "resid" -> adds into ``resid`` [M, N]
     float32 in place and returns ``(ss, xw)`` of the new stream for the norm whose weight is
-    ``next_weight`` (``(None, None)`` without it).
+    ``next_weight`` (``(None, None)`` without it).  ``xielu`` [2] float32 (see :func:`xielu`), with the epilogue "bf16":
+    the output passes the activation before it is rounded.
     """
-    _cuda(weight, act, xw, ss_in, bias, resid, next_weight)
+    _cuda(weight, act, xw, ss_in, bias, resid, next_weight, xielu)
+    _f32(xielu, "the activation's numbers")
     N, K = weight.shape
     pro = "act" if act is not None else "norm"
     src = act if act is not None else xw
@@ -360,7 +389,7 @@ def skinny_linear(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None,
     _check(lib, lib.vapi_skinny_linear(
         _p(weight), N, K, M, _PRO[pro], _p(act), _p(xw), _p(ss_in), 0 if ss_in is None else ss_in.shape[0],
         ctypes.c_float(eps), _EPI[epilogue], _p(out_bf16), _p(out_f32), ctypes.c_longlong(out_stride), _p(bias),
-        _p(resid), _p(sso), _p(next_weight), _p(xwo), rpb, _stream()))
+        _p(resid), _p(sso), _p(next_weight), _p(xwo), rpb, _stream(), _p(xielu)))
     if epilogue == "resid":
         return sso, xwo
     return out_bf16 if out_bf16 is not None else out_f32
@@ -440,9 +469,10 @@ def _tc_plan(N: int, K: int, M: int, epi: int):
 
 
 def _fused_product(which: str, weight: torch.Tensor, act, xw, ss_in, eps: float, epilogue: str, bias, resid,
-                   next_weight, status):
+                   next_weight, status, xielu=None):
     """Operand checks, outputs and the call shared by :func:`linear_tc` and :func:`prompt_linear`."""
-    _cuda(weight, act, xw, ss_in, bias, resid, next_weight)
+    _cuda(weight, act, xw, ss_in, bias, resid, next_weight, xielu)
+    _f32(xielu, "the activation's numbers")
     N, K = weight.shape
     pro = "act" if act is not None else "norm"
     src = act if act is not None else xw
@@ -487,7 +517,7 @@ def _fused_product(which: str, weight: torch.Tensor, act, xw, ss_in, eps: float,
     _check(lib, fn(
         _p(weight), N, K, M, _PRO[pro], _p(src), _p(ss_in), 0 if ss_in is None else ss_in.shape[0], ctypes.c_float(eps),
         _EPI[epilogue], _p(out_bf16), _p(out_f32), ctypes.c_longlong(out_stride), _p(bias), _p(resid), _p(sso),
-        _p(next_weight), _p(xwo), _p(status), _stream()))
+        _p(next_weight), _p(xwo), _p(status), _stream(), _p(xielu)))
     if epilogue == "resid":
         return sso, xwo
     return out_bf16 if out_bf16 is not None else out_f32
@@ -496,10 +526,11 @@ def _fused_product(which: str, weight: torch.Tensor, act, xw, ss_in, eps: float,
 def linear_tc(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None, xw: Optional[torch.Tensor] = None,
               ss_in: Optional[torch.Tensor] = None, eps: float = 0.0, epilogue: str = "bf16",
               bias: Optional[torch.Tensor] = None, resid: Optional[torch.Tensor] = None,
-              next_weight: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None):
+              next_weight: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None,
+              xielu: Optional[torch.Tensor] = None):
     """The tcgen05 / TMA product for 17..256 rows; same operands, epilogues and results as
     :func:`skinny_linear`."""
-    return _fused_product("linear_tc", weight, act, xw, ss_in, eps, epilogue, bias, resid, next_weight, status)
+    return _fused_product("linear_tc", weight, act, xw, ss_in, eps, epilogue, bias, resid, next_weight, status, xielu)
 
 
 #: steps of more rows than TC_MAX_ROWS go to the persistent tcgen05 product of csrc/linear_prompt.cu
@@ -542,6 +573,34 @@ def linear_swiglu(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     return swiglu(linear(x, weight))
 
 
+#: a product with xIELU behind it goes to the persistent tcgen05 product from this many rows on (0: never)
+PROMPT_XIELU_MIN_ROWS = int(os.environ.get("VAPI_PROMPT_XIELU_MIN_ROWS", "256"))
+
+
+def xielu(z: torch.Tensor, consts: torch.Tensor) -> torch.Tensor:
+    """The xIELU activation elementwise, ``consts`` = [up, down] float32 on the device: ``up z^2 + z / 2`` for z > 0,
+    ``down (exp(z) - 1 - z) + z / 2`` for z <= 0."""
+    _cuda(z, consts)
+    _contig(z, "activations")
+    _f32(consts, "the activation's numbers")
+    out = torch.empty_like(z)
+    lib = _lib("elementwise")
+    _check(lib, lib.vapi_xielu(_p(z), _p(out), _dt(z), _p(consts), ctypes.c_longlong(z.numel()), _stream()))
+    return out
+
+
+def linear_xielu(x: torch.Tensor, weight: torch.Tensor, consts: torch.Tensor) -> torch.Tensor:
+    """``xielu(x @ W.T)``: the activation rides on the product wherever one of this package's own kernels takes it (decode
+    steps, prompt-sized bfloat16 steps), else it is a kernel behind the library's product."""
+    rows = x.shape[0]
+    if x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and x.is_contiguous() and weight.is_contiguous():
+        if rows <= TC_MAX_ROWS and few_rows_applies(rows, weight):
+            return few_rows_linear(weight, act=x, epilogue="bf16", xielu=consts)
+        if 0 < PROMPT_XIELU_MIN_ROWS <= rows and rows > TC_MAX_ROWS and weight.shape[0] % 8 == 0 and weight.shape[1] % 8 == 0:
+            return prompt_linear(weight, act=x, epilogue="bf16", xielu=consts)
+    return xielu(linear(x, weight), consts)
+
+
 def prompt_force(bn: int = 0, pair: int = 0) -> None:
     """Fix the tile (128 | 256 features) and the blocks working on a tile (1 | 2) of
     :func:`prompt_linear` for the calls that follow; 0 gives the choice back to the kernel's plan."""
@@ -552,10 +611,11 @@ def prompt_force(bn: int = 0, pair: int = 0) -> None:
 def prompt_linear(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None, xw: Optional[torch.Tensor] = None,
                   ss_in: Optional[torch.Tensor] = None, eps: float = 0.0, epilogue: str = "bf16",
                   bias: Optional[torch.Tensor] = None, resid: Optional[torch.Tensor] = None,
-                  next_weight: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None):
+                  next_weight: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None,
+                  xielu: Optional[torch.Tensor] = None):
     """The persistent tcgen05 / TMA product for prompt-sized steps; same operands, epilogues and
     results as :func:`skinny_linear`."""
-    return _fused_product("linear_prompt", weight, act, xw, ss_in, eps, epilogue, bias, resid, next_weight, status)
+    return _fused_product("linear_prompt", weight, act, xw, ss_in, eps, epilogue, bias, resid, next_weight, status, xielu)
 
 
 def few_rows_applies(rows: int, weight: torch.Tensor) -> bool:
@@ -1110,16 +1170,68 @@ def scaled_add_rmsnorm(x: torch.Tensor, y1: Optional[torch.Tensor], s1: Optional
     return out
 
 
+#: how many tokens a block of :func:`shift_add_rmsnorm` takes one after another in steps of many tokens (the row before
+#: a block's first one is worked out twice)
+SHIFT_ROWS = int(os.environ.get("VAPI_SHIFT_ROWS", "4"))
+
+
+def shift_add_rmsnorm(x: torch.Tensor, y1: Optional[torch.Tensor], s1: Optional[torch.Tensor], y2: Optional[torch.Tensor],
+                      s2: Optional[torch.Tensor], weight: torch.Tensor, eps: float, shift: torch.Tensor, state: torch.Tensor,
+                      state_slots: torch.Tensor, tok_seq: torch.Tensor, cu_q: torch.Tensor, positions: torch.Tensor,
+                      out_dtype: torch.dtype, plain: bool = True, status: Optional[torch.Tensor] = None):
+    """:func:`scaled_add_rmsnorm` with a token shift behind the norm: ``v = x + s1 * y1 + s2 * y2``,
+    ``h = rmsnorm(v) * weight`` and ``shifted_t = h_t + (h_{t-1} - h_t) * shift`` with the previous token's h of the same
+    sequence (zeros at position 0), all float32 until the stores.  ``state`` [slots, >= H] float32 holds each request's
+    last h and is moved on.  Returns ``(v, h, shifted)``: the new stream (x itself when nothing was pending; x is never
+    written) and both rows in ``out_dtype``; ``plain`` False leaves h out (None)."""
+    _cuda(x, y1, s1, y2, s2, weight, shift, state, state_slots, tok_seq, cu_q, positions)
+    for t, w in ((x, "residual stream"), (s1, "layer scale"), (s2, "layer scale"), (weight, "norm weight"), (shift, "token shift")):
+        _f32(t, w)
+    for t, w in ((state_slots, "state slots"), (tok_seq, "tok_seq"), (cu_q, "cu_q"), (positions, "positions")):
+        _i32(t, w)
+    n, hidden = x.shape
+    for y in (y1, y2):
+        if y is not None:
+            _contig(y, "sublayer output")
+            if y.shape != x.shape or y.dtype != out_dtype:
+                raise KernelError("a sublayer's output must have the stream's shape and the activation dtype")
+    for v in (s1, s2, weight, shift):
+        if v is not None and v.numel() != hidden:
+            raise KernelError(f"scales, norm weights and shifts must have {hidden} elements")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < hidden:
+        raise KernelError(f"the state must be float32 [slots, >= {hidden}] with unit inner stride")
+    if y1 is None and y2 is not None:
+        y1, s1, y2, s2 = y2, s2, None, None
+    new = torch.empty_like(x) if y1 is not None else x
+    h = torch.empty((n, hidden), dtype=out_dtype, device=x.device) if plain else None
+    shifted = torch.empty((n, hidden), dtype=out_dtype, device=x.device)
+    rows = SHIFT_ROWS if n >= 4 * sm_count() else 1
+    lib = _lib("elementwise")
+    _check(lib, lib.vapi_shift_add_rmsnorm(
+        _p(x), _p(y1), _p(s1), _p(y2), _p(s2), _p(weight), ctypes.c_float(eps), _p(shift), _p(positions), _p(tok_seq), _p(cu_q),
+        _p(state_slots), _p(state), ctypes.c_longlong(state.stride(0)), state.shape[0], _p(new if y1 is not None else None),
+        _p(h), _p(shifted), _DT[out_dtype], n, hidden, rows, _p(status), _stream()))
+    return new, h, shifted
+
+
 def latent_prepare(down: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, q_weight: Optional[torch.Tensor],
                    kv_weight: torch.Tensor, eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot: int,
                    cache_layer: Optional[torch.Tensor], page_size: int, slot_mapping: Optional[torch.Tensor],
-                   out_dtype: torch.dtype, status: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                   out_dtype: torch.dtype, status: Optional[torch.Tensor] = None, interleaved: bool = False,
+                   q: Optional[torch.Tensor] = None, qfull: Optional[torch.Tensor] = None, heads: int = 0,
+                   dim: int = 0) -> Optional[torch.Tensor]:
     """Latent attention's cache write.  ``down`` [n, >= q_rank + kv_rank + rot_dim] float32 holds a token's three
     down-projections.  Returns the query latent ``rmsnorm(down[:, :q_rank]) * q_weight`` [n, q_rank] in ``out_dtype``
     (None for ``q_rank`` 0) and writes ``rmsnorm(latent) * kv_weight | rotate(key part)`` as the token's row of
     ``cache_layer``, flat pages [pages, page_size * (kv_rank + rot_dim)].  The rotation pairs element i with
-    i + rot/2 over the first ``rot`` elements of the key part; ``cos``/``sin`` [n, rot/2] float32."""
-    _cuda(down, q_weight, kv_weight, cos, sin, cache_layer, slot_mapping)
+    i + rot/2 (``interleaved``: 2i with 2i + 1) over the first ``rot`` elements of the key part; ``cos``/``sin``
+    [n, rot/2] float32.  With ``q`` and ``qfull`` (and ``q_rank`` 0) the work of :func:`latent_rotate_q` on ``heads``
+    queries of ``dim`` unrotated elements rides on the same kernel."""
+    _cuda(down, q_weight, kv_weight, cos, sin, cache_layer, slot_mapping, q, qfull)
+    if q is not None:
+        _latent_queries(q, qfull, down.shape[0], heads, dim, rot_dim, kv_rank)
+        if q.dtype != out_dtype or q_rank > 0:
+            raise KernelError("queries that ride along have the activation dtype and no latent of their own")
     _f32(q_weight, "query latent norm weight")
     _f32(kv_weight, "latent norm weight")
     _f32(cos, "cos")
@@ -1144,26 +1256,33 @@ def latent_prepare(down: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, 
     _check(lib, lib.vapi_latent_prepare(_p(down), ctypes.c_longlong(down.stride(0)), _p(q_weight), _p(kv_weight),
                                         ctypes.c_float(eps), _p(cos), _p(sin), int(rot), _p(cq), _p(cache_layer),
                                         _DT[out_dtype], _p(slot_mapping), n, int(q_rank), int(kv_rank), int(rot_dim),
-                                        int(page_size), num_pages, _p(status), _stream()))
+                                        int(page_size), num_pages, _p(status), _stream(), 1 if interleaved else 0, _p(q),
+                                        ctypes.c_longlong(q.stride(0) if q is not None else 0), _p(qfull), int(heads), int(dim)))
     return cq
 
 
+def _latent_queries(q, qfull, n, heads, dim, rot_dim, kv_rank) -> None:
+    _contig(qfull, "attention queries")
+    if (q.dtype != qfull.dtype or q.dim() != 2 or q.shape[0] != n or q.shape[1] < heads * (dim + rot_dim) or q.stride(1) != 1
+            or qfull.numel() != n * heads * (kv_rank + rot_dim)):
+        raise KernelError("queries of one dtype, [n, heads * (dim + rot_dim)] and [n, heads, kv_rank + rot_dim]")
+
+
 def latent_rotate_q(q: torch.Tensor, qfull: torch.Tensor, heads: int, dim: int, rot_dim: int, kv_rank: int,
-                    cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot: int) -> None:
+                    cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot: int, interleaved: bool = False) -> None:
     """The rotated part of every head's query, ``q`` [n, heads * (dim + rot_dim)], rotated by the token's position
     into the last ``rot_dim`` columns of ``qfull`` [n, heads, kv_rank + rot_dim] (contiguous)."""
     _cuda(q, qfull, cos, sin)
     _f32(cos, "cos")
     _f32(sin, "sin")
-    _contig(qfull, "attention queries")
     n = q.shape[0]
-    if q.dtype != qfull.dtype or q.stride(1) != 1 or qfull.numel() != n * heads * (kv_rank + rot_dim):
-        raise KernelError("queries of one dtype, [n, heads * (dim + rot_dim)] and [n, heads, kv_rank + rot_dim]")
+    _latent_queries(q, qfull, n, heads, dim, rot_dim, kv_rank)
     if rot > 0 and (cos is None or sin is None or cos.shape != (n, rot // 2) or sin.shape != cos.shape):
         raise KernelError("cos/sin must be [n, rot/2]")
     lib = _lib("latent")
     _check(lib, lib.vapi_latent_rotate_q(_p(q), ctypes.c_longlong(q.stride(0)), _p(cos), _p(sin), int(rot), _p(qfull), _dt(q),
-                                         n, int(heads), int(dim), int(rot_dim), int(kv_rank), _stream()))
+                                         n, int(heads), int(dim), int(rot_dim), int(kv_rank), _stream(),
+                                         1 if interleaved else 0))
 
 
 def head_products(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -1184,24 +1303,35 @@ def head_products(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] 
 def latent_attention(q: torch.Tensor, cache_layer: torch.Tensor, page_size: int, block_table: torch.Tensor, cu_q: torch.Tensor,
                      seqlens_k: torch.Tensor, n: int, num_seqs: int, max_q: int, max_k: int, heads: int, kv_rank: int,
                      rot_dim: int, scale: float, *, splits: Optional[int] = None,
-                     status: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     status: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of ``heads`` query heads over one cached row per token, ``[latent (kv_rank) | rotated key part
     (rot_dim)]``: a score is ``scale * q . row`` over the whole row and a head's output is the softmax-weighted sum of
     the rows' latents, so keys and values are the same memory.  ``q`` [n, heads * (kv_rank + rot_dim)] contiguous;
-    ``cache_layer`` flat pages [pages, page_size * (kv_rank + rot_dim)]; returns [n, heads * kv_rank]."""
+    ``cache_layer`` flat pages [pages, page_size * (kv_rank + rot_dim)]; ``sinks`` as for :func:`masked_attention`;
+    returns [n, heads * kv_rank]."""
     width = kv_rank + rot_dim
     _contig(q, "queries")
     return masked_attention(q, heads * width, cache_layer, page_size, block_table, cu_q, seqlens_k, n, num_seqs, max_q, max_k,
-                            heads, 1, width, kv_rank, scale, splits=splits, status=status, shared_kv=True)
+                            heads, 1, width, kv_rank, scale, splits=splits, status=status, shared_kv=True, sinks=sinks)
+
+
+def _output(out: Optional[torch.Tensor], shape, dtype: torch.dtype, device) -> torch.Tensor:
+    """The tensor a kernel writes: a new one, or the given one if it fits (rows may be parts of wider rows)."""
+    if out is None:
+        return torch.empty(shape, dtype=dtype, device=device)
+    if tuple(out.shape) != tuple(shape) or out.dtype != dtype or out.stride(1) != 1 or not out.is_cuda:
+        raise KernelError(f"the given output must be {tuple(shape)} {dtype} on the device with unit inner stride")
+    return out
 
 
 def gated_group_rmsnorm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, group: int,
-                        gate_first: bool, out_dtype: torch.dtype, gate: str = "silu") -> torch.Tensor:
+                        gate_first: bool, out_dtype: torch.dtype, gate: str = "silu",
+                        out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """RMS norm over equal groups of ``group`` columns of the float32 rows ``y`` [n, width] with a
     SiLU gate ``z`` [n, width] (any row stride): ``norm(y) * weight * silu(z)``, or with
     ``gate_first`` ``norm(y * silu(z)) * weight``.  ``weight`` is indexed by column modulo its
     length (one weight per group member, or one per column).  ``gate`` "sigmoid" puts ``sigmoid(z)`` where
-    ``silu(z)`` stands."""
+    ``silu(z)`` stands.  ``out`` may be given: [n, width] with unit inner stride, e.g. a part of a wider buffer."""
     if gate not in ("silu", "sigmoid"):
         raise KernelError(f"gate `{gate}` is not one of silu, sigmoid")
     _cuda(y, z, weight)
@@ -1210,12 +1340,12 @@ def gated_group_rmsnorm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, 
     n, width = y.shape
     if z.shape != y.shape or z.stride(1) != 1 or z.dtype != out_dtype:
         raise KernelError("the gate must be [n, width] of the activation dtype with unit inner stride")
-    out = torch.empty((n, width), dtype=out_dtype, device=y.device)
+    out = _output(out, (n, width), out_dtype, y.device)
     lib = _lib("elementwise")
     _check(lib, lib.vapi_gated_group_rmsnorm(_p(y), _p(z), ctypes.c_longlong(z.stride(0)), _dt(z), _p(weight),
                                              weight.numel(), ctypes.c_float(eps),
                                              (1 if gate_first else 0) | (2 if gate == "sigmoid" else 0), _p(out), n, width,
-                                             int(group), _stream()))
+                                             int(group), _stream(), ctypes.c_longlong(out.stride(0))))
     return out
 
 
@@ -1305,7 +1435,9 @@ def masked_attention(q: torch.Tensor, q_row_stride: int, cache_layer: torch.Tens
                      max_q: int, max_k: int, nh: int, nkv: int, dk: int, dv: int, scale: float, *, window: int = 0,
                      chunk: int = 0, sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                      splits: Optional[int] = None, status: Optional[torch.Tensor] = None, keep: int = 0,
-                     shared_kv: bool = False) -> torch.Tensor:
+                     shared_kv: bool = False, weights: str = "softmax", softcap: float = 0.0,
+                     score_bias: Optional[torch.Tensor] = None, out_scale: float = 1.0,
+                     out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal GQA attention of a mixed batch over the paged cache for keys of width ``dk`` and values
     of width ``dv``; returns [n, nh*dv].  A query at position p sees key i iff i <= p, (i > p - window or
     i < keep) (``window`` > 0; ``keep``: the first tokens of a sequence, which a window never leaves behind)
@@ -1313,8 +1445,16 @@ def masked_attention(q: torch.Tensor, q_row_stride: int, cache_layer: torch.Tens
     exp(sink_h) to head h's softmax denominator; ``gate`` [n, nh] (any row stride) multiplies head
     h's output by sigmoid(gate).  ``cache_layer``: flat pages as for :func:`qk_norm_rope_write_split`.
     ``shared_kv``: a page holds key rows alone, [nkv, page_size, dk], and a key's value is the first ``dv`` elements
-    of its own row (latent attention)."""
-    _cuda(q, cache_layer, block_table, cu_q, seqlens_k, sinks, gate)
+    of its own row (latent attention).  ``softcap`` > 0: a score passes ``softcap * tanh(score / softcap)``;
+    ``score_bias`` [nh] float32 is added to head h's scores behind the cap; ``weights`` "sigmoid": a visible key's weight
+    is the sigmoid of its score and nothing is normalised over the keys (no sink then).  The output is multiplied by
+    ``out_scale`` and may go into ``out`` [n, nh*dv] with unit inner stride, e.g. a part of a wider buffer."""
+    _cuda(q, cache_layer, block_table, cu_q, seqlens_k, sinks, gate, score_bias)
+    _f32(score_bias, "score bias")
+    if weights not in ("softmax", "sigmoid"):
+        raise KernelError(f"attention weights `{weights}` are not one of softmax, sigmoid")
+    if (score_bias is not None and score_bias.numel() != nh) or (weights == "sigmoid" and sinks is not None):
+        raise KernelError("one score bias per head is needed, and sigmoid weights have no sink")
     _i32(block_table, "block table")
     _i32(cu_q, "cu_q")
     _i32(seqlens_k, "seqlens_k")
@@ -1341,7 +1481,7 @@ def masked_attention(q: torch.Tensor, q_row_stride: int, cache_layer: torch.Tens
         if chunk > 0:
             keys = min(keys, chunk + max_q - 1)
         splits = masked_attention_splits(num_seqs, max_q, keys, nh, nkv)
-    out = torch.empty((n, nh * dv), dtype=q.dtype, device=q.device)
+    out = _output(out, (n, nh * dv), q.dtype, q.device)
     part_o = part_ml = None
     if splits > 1:
         part_o = torch.empty((n * nh * splits * dv,), dtype=torch.float32, device=q.device)
@@ -1351,7 +1491,8 @@ def masked_attention(q: torch.Tensor, q_row_stride: int, cache_layer: torch.Tens
         _p(q), ctypes.c_longlong(q_row_stride), _p(cache_layer), _dt(q), _p(block_table), block_table.stride(0), _p(cu_q),
         _p(seqlens_k), _p(sinks), _p(gate), ctypes.c_longlong(gate_stride), _p(out), _p(part_o), _p(part_ml), n, num_seqs,
         max_q, nh, nkv, dk, dv, int(page_size), cache_layer.shape[0], ctypes.c_float(scale), int(window), int(chunk),
-        int(splits), _p(status), _stream(), int(keep), 1 if shared_kv else 0),
+        int(splits), _p(status), _stream(), int(keep), 1 if shared_kv else 0, ctypes.c_float(softcap),
+        1 if weights == "sigmoid" else 0, _p(score_bias), ctypes.c_float(out_scale), ctypes.c_longlong(out.stride(0))),
         2 if splits > 1 or (not shared_kv and q.dtype == torch.bfloat16 and dk == dv == 64 and max_q >= 64 and num_seqs > 1) else 1)
     return out
 

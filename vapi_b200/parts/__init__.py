@@ -1,5 +1,5 @@
 """Parts a model is assembled from: mixers, feed-forwards, norms, position encodings, blocks."""
-from .base import (CacheView, FeedForward, Mixer, Norm, NormedStream, PagedBuffer, PagedSpec, PostNormed, ScaledPair, StreamState, Part, PositionEncoding, StateSpec,
+from .base import (CacheView, FeedForward, Mixer, Norm, NormedStream, PagedBuffer, PagedSpec, PostNormed, ProjectedForm, ScaledPair, StreamState, Part, PositionEncoding, StateSpec,
                    TensorSpec, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, make_part,
                    register_feed_forward, register_mixer, register_norm, register_position_encoding)
 from .norm import LayerNorm, NoNorm, RMSNorm
@@ -7,7 +7,7 @@ from .rope import RotaryEncoding, ScaledRotaryEncoding
 from .attention import GQAttention
 from .shortconv import ShortConv
 from .recurrent import GatedDeltaMixer, Mamba2Mixer, RGLRUMixer
-from .feedforward import SwiGLU
+from .feedforward import SwiGLU, XIELU
 from .moe import SparseMoE
 from .embedding import OutputHead, TokenEmbedding
 from .block import BLOCKS, ParallelBlock, PreNormBlock, SandwichBlock, register_block
@@ -25,4 +25,5 @@ __all__ = [
     "TokenEmbedding", "PreNormBlock", "SandwichBlock", "PostNormed", "ScaledRotaryEncoding", "GatedDeltaMixer", "Mamba2Mixer",
     "LayerNorm", "RGLRUMixer", "SparseMoE", "HyperBlock", "HyperPending", "ParallelMixer",
     "NoNorm", "MatrixMemoryMixer", "GatedLinearAttentionMixer", "ParallelBlock", "ScaledPair", "LatentAttention", "StreamInjection",
+    "ProjectedForm", "XIELU",
 ]

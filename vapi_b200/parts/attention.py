@@ -7,7 +7,7 @@ from typing import Any, Dict, List, Optional
 import torch
 
 from .. import ops
-from .base import CacheView, Mixer, PagedBuffer, PagedSpec, StreamState, TensorSpec, register_mixer
+from .base import CacheView, Mixer, PagedBuffer, PagedSpec, ProjectedForm, StreamState, TensorSpec, register_mixer
 
 
 class GQAttention(Mixer):
@@ -34,8 +34,11 @@ class GQAttention(Mixer):
     "interleaved": pairs (2i, 2i+1)) and ``weight_suffix`` (what follows a projection's name in the
     checkpoint), ``bias_suffix`` (what follows it for its bias), ``fixed_sink`` (a sink whose score is this number
     for every head, with no tensor: 0.0 puts a plain one into the denominator) and ``q_temp`` = (coef, every) (the
-    query at position p is multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``).  Any of these but the
-    suffixes sends the mixer to the general kernels
+    query at position p is multiplied by ``1 + coef * ln(floor((p + 1) / every) + 1)``), ``qk_norm_weight`` False (the
+    q/k norms have no weight, so that norm and rotation may change places), ``softcap`` (a score passes
+    ``cap * tanh(score / cap)``), ``weights`` "sigmoid" (a visible key's weight is the sigmoid of its score, and nothing
+    is normalised over the keys) and ``score_bias`` (a stored number per head is added to the score behind the cap).
+    Any of these but the suffixes sends the mixer to the general kernels
     (``ops.qk_norm_rope_write_split``, ``ops.masked_attention``); the plain form keeps the
     specialised ones.
     """
@@ -47,7 +50,8 @@ class GQAttention(Mixer):
                  v_head_dim: Optional[int] = None, chunk: int = 0, sink: bool = False, head_gate: bool = False,
                  rope_layout: str = "half", weight_suffix: str = ".weight", keep_first: int = 0, out_gate: bool = False,
                  qk_norm: str = "head", bias_suffix: str = ".bias", fixed_sink: Optional[float] = None,
-                 q_temp: Optional[Any] = None):
+                 q_temp: Optional[Any] = None, qk_norm_weight: bool = True, softcap: Optional[float] = None,
+                 weights: str = "softmax", score_bias: bool = False):
         if n_heads <= 0 or n_kv_heads <= 0 or n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads are not a multiple of {n_kv_heads} kv heads")
         if rope_layout not in ("half", "interleaved"):
@@ -67,9 +71,18 @@ class GQAttention(Mixer):
         self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp is not None else None
         if self.q_temp is not None and (self.q_temp[1] < 1 or self.whole_norm):
             raise ValueError("a query temperature needs `every` >= 1 and q/k norms per head")
+        if weights not in ("softmax", "sigmoid"):
+            raise ValueError(f"attention weights `{weights}` are not one of softmax, sigmoid")
+        self.weights, self.softcap, self.score_bias = weights, float(softcap) if softcap else 0.0, bool(score_bias)
+        if weights == "sigmoid" and (self.sink or fixed_sink is not None):
+            raise ValueError("a sink belongs to a softmax")
+        self.qk_norm_weight = bool(qk_norm_weight)
+        if not self.qk_norm_weight and self.whole_norm:
+            raise ValueError("q/k norms without a weight run per head")
         self.general = bool(self.dv != int(head_dim) or self.chunk > 0 or self.sink or self.head_gate or self.interleaved
                             or self.keep_first > 0 or self.out_gate or self.whole_norm or self.fixed_sink is not None
-                            or self.q_temp is not None)
+                            or self.q_temp is not None or weights != "softmax" or self.softcap > 0 or self.score_bias
+                            or not self.qk_norm_weight)
         if self.general:
             if head_dim % 4 or self.dv % 4 or not (4 <= head_dim <= 256 and 4 <= self.dv <= 256):
                 raise ValueError(f"head sizes {head_dim} / {self.dv} must be multiples of 4 in 4..256")
@@ -84,10 +97,10 @@ class GQAttention(Mixer):
         self.bias = bool(bias)
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(self.d)
         self.names = {"q": "q_proj", "k": "k_proj", "v": "v_proj", "o": "out_proj",
-                      "q_norm": "q_layernorm", "k_norm": "k_layernorm", "sink": "sinks", "gate": "gate_proj"}
+                      "q_norm": "q_layernorm", "k_norm": "k_layernorm", "sink": "sinks", "gate": "gate_proj", "score_bias": "score_bias"}
         if names:
             self.names.update(names)
-        self.w_qkv = self.b_qkv = self.w_o = self.b_o = self.q_w = self.k_w = self.sinks = None
+        self.w_qkv = self.b_qkv = self.w_o = self.b_o = self.q_w = self.k_w = self.sinks = self.bias_h = None
 
     def cache_spec(self):
         # (for equal widths this is PagedSpec.kv: keys [nkv, page, d], then values [nkv, page, dv])
@@ -105,13 +118,15 @@ class GQAttention(Mixer):
             specs.append(TensorSpec(f"{prefix}{n['gate']}{x}", (nh if self.head_gate else nh * self.dv, h)))
         if self.sink:
             specs.append(TensorSpec(f"{prefix}{n['sink']}", (nh,), role="vector", init="normal"))
+        if self.score_bias:
+            specs.append(TensorSpec(f"{prefix}{n['score_bias']}", (nh,), role="vector", init="normal"))
         if self.bias:
             b = self.bsfx
             specs += [TensorSpec(f"{prefix}{n['q']}{b}", (nh * d,), role="vector"),
                       TensorSpec(f"{prefix}{n['k']}{b}", (nkv * d,), role="vector"),
                       TensorSpec(f"{prefix}{n['v']}{b}", (nkv * self.dv,), role="vector"),
                       TensorSpec(f"{prefix}{n['o']}{b}", (h,), role="vector")]
-        if self.qk_norm_eps is not None:
+        if self.qk_norm_eps is not None and self.qk_norm_weight:
             specs += [TensorSpec(f"{prefix}{n['q_norm']}{x}", (nh * d if self.whole_norm else d,), role="vector", init="ones"),
                       TensorSpec(f"{prefix}{n['k_norm']}{x}", (nkv * d if self.whole_norm else d,), role="vector", init="ones")]
         return specs
@@ -138,7 +153,11 @@ class GQAttention(Mixer):
             if self.b_qkv.numel() < self.w_qkv.shape[0]:       # the gate's rows and the padding have no bias
                 self.b_qkv = torch.cat([self.b_qkv, self.b_qkv.new_zeros(self.w_qkv.shape[0] - self.b_qkv.numel())])
             self.b_o = tensors[f"{prefix}{n['o']}{self.bsfx}"].contiguous()
-        if self.qk_norm_eps is not None:
+        if self.score_bias:
+            self.bias_h = tensors[f"{prefix}{n['score_bias']}"].contiguous()
+        if self.qk_norm_eps is not None and not self.qk_norm_weight:
+            self.q_w = self.k_w = torch.ones(self.d, dtype=torch.float32, device=self.w_o.device)
+        elif self.qk_norm_eps is not None:
             self.q_w = tensors[f"{prefix}{n['q_norm']}{x}"].contiguous()
             self.k_w = tensors[f"{prefix}{n['k_norm']}{x}"].contiguous()
 
@@ -154,6 +173,17 @@ class GQAttention(Mixer):
     def forward(self, a: torch.Tensor, ctx: Any, cache: CacheView) -> torch.Tensor:
         qkv = ops.linear(a, self.w_qkv, self.b_qkv)
         return ops.linear(self._attend(qkv, ctx, cache), self.w_o, self.b_o)
+
+    def pieces(self):
+        if not self.general or self.out_gate:
+            return None
+        return ProjectedForm(self.w_qkv, self.b_qkv, self.w_o, self.b_o, first=True)
+
+    def inner(self, h, at, ctx, cache, out, scale):
+        if at != 0:
+            raise ValueError("q, k and v lead the rows of their product")
+        cos, sin = ctx.pos[self.pos] if self.pos is not None else (None, None)
+        self._attend_general(h, ctx, cache, cos, sin, out, scale)
 
     def forward_stream(self, a, ctx, cache, x, next_weight):
         n = x.shape[0]
@@ -198,8 +228,9 @@ class GQAttention(Mixer):
         return y
 
 
-    def _attend_general(self, qkv, ctx, cache, cos, sin):
-        """Unlike key and value widths, a chunked mask, a sink, a head gate or interleaved pairs."""
+    def _attend_general(self, qkv, ctx, cache, cos, sin, out=None, scale: float = 1.0):
+        """Unlike key and value widths, a chunked mask, a sink, a head gate, interleaved pairs or sigmoid weights; ``scale``
+        times the result, into ``out`` when given.  Columns of ``qkv`` behind q, k, v and the gate are left alone."""
         nh, nkv, d, dv = self.nh, self.nkv, self.d, self.dv
         grp = cache.group
         pages = cache.tensor                                    # flat [pages, page_size * nkv * (d + dv)]
@@ -218,8 +249,12 @@ class GQAttention(Mixer):
         y = ops.masked_attention(qkv, qkv.stride(0), pages, page_size, grp.block_table, ctx.cu_q, ctx.seqlens_k,
                                  ctx.n, ctx.num_seqs, ctx.max_q, max_k, nh, nkv, d, dv, self.scale,
                                  window=self.window, chunk=self.chunk, sinks=self.sinks, gate=gate, splits=splits,
-                                 status=ctx.status, keep=self.keep_first)
+                                 status=ctx.status, keep=self.keep_first, weights=self.weights, softcap=self.softcap,
+                                 score_bias=self.bias_h, out_scale=1.0 if self.out_gate else scale,
+                                 out=None if self.out_gate else out)
         if self.out_gate:
+            if out is not None or scale != 1.0:
+                raise ValueError("a gate as wide as the heads' output has no form that writes into a wider buffer")
             off = (nh + nkv) * d + nkv * dv
             y = ops.sigmoid_gate(y, qkv[:, off:off + nh * dv])
         return y

@@ -121,7 +121,8 @@ class CacheView:
     group.  ``state``: ``tensor`` is this call site's view [slots, *shape]; ``ctx.state_slots``
     [S] names each sequence's slot.  ``write`` False: the call site reads a cache another layer
     owns.  ``multi``: the mixer is several mixers side by side (its ``cache_spec`` is a tuple); ``parts`` holds one
-    view per member, in the order of :meth:`Mixer.members`.
+    view per member, in the order of :meth:`Mixer.members`.  ``block``: the view of what the *block* around the mixer
+    keeps for itself (:meth:`Part.block_cache_spec`); it belongs to the call site whatever ``write`` says.
     """
 
     kind: str                 # "paged" | "state" | "none" | "multi"
@@ -131,6 +132,7 @@ class CacheView:
     buffers: Optional[Dict[str, torch.Tensor]] = None
     spec: Any = None
     parts: Optional[List["CacheView"]] = None
+    block: Optional["CacheView"] = None
 
     def stacked(self) -> torch.Tensor:
         """Buffers of one shape as a single tensor [pages, n_buffers, rows, page_size, width]."""
@@ -194,6 +196,18 @@ class ScaledPair:
     scale_b: Optional[torch.Tensor] = None
 
 
+@dataclass
+class ProjectedForm:
+    """The projections of a mixer ``W_out inner(W_in a + b_in) + b_out`` (:meth:`Mixer.pieces`).  ``first``: the inner
+    part only works on the leading columns of its product's rows (it rewrites them in place, row by row)."""
+
+    w_in: torch.Tensor
+    b_in: Optional[torch.Tensor]
+    w_out: torch.Tensor
+    b_out: Optional[torch.Tensor]
+    first: bool = False
+
+
 # --------------------------------------------------------------------------------------
 # the parts
 
@@ -206,6 +220,12 @@ class Part:
 
     def bind(self, tensors: Dict[str, torch.Tensor], prefix: str, dtype: torch.dtype) -> None:
         """Take the loaded tensors (by full checkpoint name); fuse or reshape them once."""
+
+    def block_cache_spec(self) -> Optional[StateSpec]:
+        """What a block, or the embedding, keeps per request besides what its mixer asks for (None: nothing).  Every call
+        site has its own, also one whose mixer reads another call site's cache.  A block gets it as ``cache.block``,
+        the embedding as ``cache``."""
+        return None
 
 
 class Norm(Part):
@@ -262,6 +282,17 @@ class Mixer(Part):
         fixed-shape (captured) decode step, whose kernels cannot follow the batch's real lengths;
         the answer comes back to the mixer as ``cache.group.splits``.  1: no cutting."""
         return 1
+
+    # A mixer of the form ``W_out inner(W_in a + b_in) + b_out`` may offer itself in pieces, so that a mixer made of
+    # several can run all in-projections as one product and all out-projections as another:
+    def pieces(self) -> Optional["ProjectedForm"]:
+        """This (bound) mixer's projections, or None if it is not of that form."""
+        return None
+
+    def inner(self, h: torch.Tensor, at: int, ctx: "Any", cache: CacheView, out: torch.Tensor, scale: float) -> None:
+        """What lies between the projections: reads columns ``at ..`` of ``h`` [n, columns], writes ``scale`` times the
+        out-projection's input into ``out`` [n, its width] (unit inner stride, rows of a wider buffer)."""
+        raise NotImplementedError
 
     def forward_stream(self, a: NormedStream, ctx: "Any", cache: CacheView, x: torch.Tensor,
                        next_weight: torch.Tensor):

@@ -5,7 +5,7 @@ from typing import Any, Callable, Dict, List, Optional
 
 import torch
 
-from .base import CacheView, FeedForward, Mixer, Norm, Part, PostNormed, ScaledPair, StreamState, TensorSpec
+from .base import CacheView, FeedForward, Mixer, Norm, Part, PostNormed, ScaledPair, StateSpec, StreamState, TensorSpec
 
 BLOCKS: Dict[str, Callable[..., "Part"]] = {}
 
@@ -147,16 +147,30 @@ class ParallelBlock(Part):
     Neither output is added by a kernel of its own: the block hands both on as a :class:`ScaledPair`, and the norm
     that reads the stream next (the next block's, or the model's final norm) scales and adds them while it reads
     the row.  ``sub`` gives the checkpoint sub-prefix of ``norm``, ``mixer`` and ``ffn``.
+
+    ``shift`` names a vector over the width (token shift): the mixer then reads ``h_t + (h_{t-1} - h_t) * shift`` with
+    the previous token's h (zeros at position 0), the feed-forward h as it is.  The last h of a request is a float32
+    state of the block's own.  The norm (an RMS norm), what is pending for the stream and the shift are one kernel; it
+    puts the new stream into memory of its own, so such a block's ``forward`` returns ``(stream, pending)``
+    (``replaces_stream``).
     """
 
     def __init__(self, norm: Norm, mixer: Mixer, ffn: Optional[FeedForward], sub: Dict[str, str],
-                 scales=(None, None), hidden: Optional[int] = None):
+                 scales=(None, None), hidden: Optional[int] = None, shift: Optional[str] = None):
         self.norm, self.mixer, self.ffn, self.sub = norm, mixer, ffn, dict(sub)
         self.scale_names = (scales[0], scales[1] if ffn is not None else None)
         self.hidden = int(hidden) if hidden is not None else int(getattr(norm, "dim", 0))
-        if any(self.scale_names) and self.hidden <= 0:
-            raise ValueError("a layer scale needs the width")
-        self.s_m = self.s_f = None
+        if (any(self.scale_names) or shift) and self.hidden <= 0:
+            raise ValueError("a layer scale or a token shift needs the width")
+        if shift and getattr(norm, "kind", None) != "rms":
+            raise ValueError("a token shift rides on an RMS norm")
+        self.shift_name = shift
+        #: whether ``forward`` returns (stream, pending) instead of the pending output alone
+        self.replaces_stream = shift is not None
+        self.s_m = self.s_f = self.shift = None
+
+    def block_cache_spec(self):
+        return StateSpec("token_shift", (self.hidden,), torch.float32) if self.shift_name else None
 
     def _parts(self):
         out = [("norm", self.norm), ("mixer", self.mixer)]
@@ -169,6 +183,8 @@ class ParallelBlock(Part):
         for key, part in self._parts():
             out += part.tensor_specs(prefix + self.sub.get(key, ""))
         out += [TensorSpec(prefix + name, (self.hidden,), role="vector", init="ones") for name in self.scale_names if name]
+        if self.shift_name:
+            out.append(TensorSpec(prefix + self.shift_name, (self.hidden,), role="vector", init="normal"))
         return out
 
     def bind(self, tensors, prefix, dtype):
@@ -176,15 +192,33 @@ class ParallelBlock(Part):
             part.bind(tensors, prefix + self.sub.get(key, ""), dtype)
         self.s_m = tensors[prefix + self.scale_names[0]].contiguous() if self.scale_names[0] else None
         self.s_f = tensors[prefix + self.scale_names[1]].contiguous() if self.scale_names[1] else None
+        self.shift = tensors[prefix + self.shift_name].contiguous() if self.shift_name else None
 
     def first_norm(self) -> Norm:
         return self.norm
 
-    def forward(self, x: torch.Tensor, delta, ctx: Any, cache: CacheView) -> ScaledPair:
+    def forward(self, x: torch.Tensor, delta, ctx: Any, cache: CacheView):
+        if self.shift is not None:
+            return self._forward_shifted(x, delta, ctx, cache)
         h = self.norm.apply(x, delta, ctx.dtype)
         a = self.mixer.forward(h, ctx, cache)
         b = self.ffn.forward(h, ctx) if self.ffn is not None else None
         return ScaledPair(a, self.s_m, b, self.s_f)
+
+    def _forward_shifted(self, x: torch.Tensor, delta, ctx: Any, cache: CacheView):
+        from .. import ops
+        if delta is None or isinstance(delta, torch.Tensor):
+            pending = (delta, None, None, None)
+        elif isinstance(delta, ScaledPair):
+            pending = (delta.a, delta.scale_a, delta.b, delta.scale_b)
+        else:
+            raise TypeError(f"a token shift cannot fold in a pending {type(delta).__name__}")
+        x, h, shifted = ops.shift_add_rmsnorm(x, *pending, self.norm.weight, self.norm.eps, self.shift, cache.block.tensor,
+                                              ctx.state_slots, ctx.tok_seq, ctx.cu_q, ctx.positions, ctx.dtype,
+                                              plain=self.ffn is not None, status=ctx.status)
+        a = self.mixer.forward(shifted, ctx, cache)
+        b = self.ffn.forward(h, ctx) if self.ffn is not None else None
+        return x, ScaledPair(a, self.s_m, b, self.s_f)
 
 
 register_block("prenorm", PreNormBlock)

@@ -1,12 +1,12 @@
 """Token embedding and the output head."""
 from __future__ import annotations
 
-from typing import Any, List, Optional
+from typing import Any, List, Optional, Tuple
 
 import torch
 
 from .. import ops
-from .base import Part, TensorSpec
+from .base import CacheView, Part, StateSpec, TensorSpec
 
 
 class TokenEmbedding(Part):
@@ -15,7 +15,8 @@ class TokenEmbedding(Part):
 
     def __init__(self, vocab: int, hidden: int, name: str = "model.embed_tokens.weight", *,
                  sinusoid_base: Optional[float] = None, streams: Optional[int] = None,
-                 position_table: Optional[str] = None, positions: int = 0, scale: float = 1.0):
+                 position_table: Optional[str] = None, positions: int = 0, scale: float = 1.0,
+                 bigram: Optional[Tuple[str, int, int, int]] = None):
         self.vocab, self.hidden, self.name = int(vocab), int(hidden), name
         #: every row is multiplied by this number (a float32 product) on its way into the stream
         self.scale = float(scale)
@@ -28,6 +29,13 @@ class TokenEmbedding(Part):
         self.position_table, self.positions = position_table, int(positions)
         if position_table is not None and self.positions <= 0:
             raise ValueError("a position table needs its number of rows")
+        #: with ``bigram`` = (tensor name, buckets, mul_prev, mul_cur) row ``(previous token * mul_prev + token * mul_cur)
+        #: mod buckets`` of that [buckets + 1, hidden] table is added (unscaled), for a sequence's first token its last row;
+        #: the previous token is then part of a request's state
+        self.bigram = (str(bigram[0]), int(bigram[1]), int(bigram[2]), int(bigram[3])) if bigram is not None else None
+        if self.bigram is not None and (self.bigram[1] <= 0 or sinusoid_base is not None or streams is not None or position_table):
+            raise ValueError("a bigram table needs a positive number of buckets, one stream and no position vectors")
+        self.bigram_table: Optional[torch.Tensor] = None
         self.table: Optional[torch.Tensor] = None
         self.freq: Optional[torch.Tensor] = None
         self.pos_rows: Optional[torch.Tensor] = None
@@ -36,19 +44,32 @@ class TokenEmbedding(Part):
         specs = [TensorSpec(self.name, (self.vocab, self.hidden))]
         if self.position_table is not None:
             specs.append(TensorSpec(self.position_table, (self.positions, self.hidden)))
+        if self.bigram is not None:
+            specs.append(TensorSpec(self.bigram[0], (self.bigram[1] + 1, self.hidden)))
         return specs
+
+    def block_cache_spec(self):
+        return StateSpec("previous_token", (1,), torch.int32) if self.bigram is not None else None
 
     def bind(self, tensors, prefix, dtype):
         self.table = tensors[self.name].contiguous()
         if self.position_table is not None:
             self.pos_rows = tensors[self.position_table].to(self.table.dtype).contiguous()
+        if self.bigram is not None:
+            self.bigram_table = tensors[self.bigram[0]].to(self.table.dtype).contiguous()
         if self.sinusoid_base is not None:
             i = torch.arange((self.hidden + 1) // 2, dtype=torch.float64)
             freq = torch.pow(torch.tensor(self.sinusoid_base, dtype=torch.float64), -2.0 * i / self.hidden)
             self.freq = freq.to(torch.float32).to(self.table.device)      # rounded once, from the exact value
 
-    def forward(self, ctx: Any, next_weight: Optional[torch.Tensor] = None):
-        """The stream; with ``next_weight`` also what a deferred norm needs: ``(x, ss, xw)``."""
+    def forward(self, ctx: Any, next_weight: Optional[torch.Tensor] = None, cache: Optional[CacheView] = None):
+        """The stream; with ``next_weight`` also what a deferred norm needs: ``(x, ss, xw)``.  ``cache``: the view of what
+        :meth:`block_cache_spec` asks for."""
+        if self.bigram is not None:
+            if next_weight is not None:
+                raise ValueError("an embedding with a bigram table has no deferred-norm form")
+            return ops.embed_bigram(self.table, self.bigram_table, ctx.tokens, ctx.positions, ctx.tok_seq, ctx.cu_q, cache.tensor,
+                                    ctx.state_slots, self.bigram[2], self.bigram[3], self.scale, ctx.status)
         if self.sinusoid_base is not None or self.streams is not None or self.pos_rows is not None:
             if next_weight is not None or self.scale != 1.0:
                 raise ValueError("an embedding with positions or several streams has no deferred-norm form and no scale")

@@ -1,4 +1,4 @@
-"""Dense SwiGLU feed-forward."""
+"""Dense feed-forwards: SwiGLU, and one hidden layer with xIELU."""
 from __future__ import annotations
 
 from typing import Any, Dict, List, Optional
@@ -63,4 +63,36 @@ class SwiGLU(FeedForward):
         return StreamState(xw, ss)
 
 
+class XIELU(FeedForward):
+    """``down(xielu(up f))`` without biases.  ``xielu(z) = a z^2 + z / 2`` for z > 0 and ``b (exp(z) - 1 - z) + z / 2`` for
+    z <= 0, with ``a = softplus(p)`` and ``b = 1/2 + softplus(q)`` from the layer's two stored numbers p, q (worked out once,
+    at bind time).  The activation is the up product's epilogue wherever one of the package's own products takes it."""
+
+    def __init__(self, hidden: int, ff: int, names: Optional[Dict[str, str]] = None, weight_suffix: str = ".weight"):
+        self.hidden, self.ff, self.sfx = int(hidden), int(ff), weight_suffix
+        self.names = {"up": "up_proj", "down": "down_proj", "act": "act"}
+        if names:
+            self.names.update(names)
+        self.w_up = self.w_down = self.act = None
+
+    def tensor_specs(self, prefix: str) -> List[TensorSpec]:
+        n = self.names
+        return [TensorSpec(f"{prefix}{n['up']}{self.sfx}", (self.ff, self.hidden)),
+                TensorSpec(f"{prefix}{n['down']}{self.sfx}", (self.hidden, self.ff)),
+                TensorSpec(f"{prefix}{n['act']}", (2,), role="vector")]
+
+    def bind(self, tensors, prefix, dtype):
+        n = self.names
+        self.w_up = tensors[f"{prefix}{n['up']}{self.sfx}"].contiguous()
+        self.w_down = tensors[f"{prefix}{n['down']}{self.sfx}"].contiguous()
+        # softplus(z) = max(z, 0) + log(1 + exp(-|z|)), rounded once from float64
+        z = tensors[f"{prefix}{n['act']}"].to(torch.float64)
+        sp = torch.clamp(z, min=0.0) + torch.log1p(torch.exp(-z.abs()))
+        self.act = torch.stack([sp[0], 0.5 + sp[1]]).to(torch.float32).contiguous()
+
+    def forward(self, f: torch.Tensor, ctx: Any) -> torch.Tensor:
+        return ops.linear(ops.linear_xielu(f, self.w_up, self.act), self.w_down)
+
+
+register_feed_forward("xielu", XIELU)
 register_feed_forward("swiglu", SwiGLU)

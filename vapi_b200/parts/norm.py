@@ -22,21 +22,23 @@ def _raw_branches(y):
 
 class RMSNorm(Norm):
     """``y = x * rsqrt(mean(x^2) + eps) * w``: the weight multiplies as it is (no ``1 + w``)
-    (crates/vapi-backend-candle/src/models/lfm2.rs:626-628).  Mean, rsqrt and the residual
-    sum are float32 whatever the activation dtype."""
+    (crates/vapi-backend-candle/src/models/lfm2.rs:626-628), unless ``offset`` says what is added to it: a weight
+    stored around zero has ``offset`` 1.  Mean, rsqrt and the residual sum are float32 whatever the activation dtype."""
 
     #: what the kernels that norm on a reader's behalf call this norm
     kind = "rms"
 
-    def __init__(self, dim: int, eps: float, weight_name: str = "weight"):
-        self.dim, self.eps, self.weight_name = int(dim), float(eps), weight_name
+    def __init__(self, dim: int, eps: float, weight_name: str = "weight", offset: float = 0.0):
+        self.dim, self.eps, self.weight_name, self.offset = int(dim), float(eps), weight_name, float(offset)
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self, prefix: str) -> List[TensorSpec]:
-        return [TensorSpec(f"{prefix}{self.weight_name}", (self.dim,), role="vector", init="ones")]
+        init = "zeros" if self.offset == 1.0 else "ones"
+        return [TensorSpec(f"{prefix}{self.weight_name}", (self.dim,), role="vector", init=init)]
 
     def bind(self, tensors: Dict[str, torch.Tensor], prefix: str, dtype: torch.dtype) -> None:
-        self.weight = tensors[f"{prefix}{self.weight_name}"].contiguous()
+        w = tensors[f"{prefix}{self.weight_name}"]
+        self.weight = (w + self.offset if self.offset else w).contiguous()
 
     def apply(self, x, delta, dtype, rows=None):
         if isinstance(delta, PostNormed):

@@ -15,7 +15,7 @@ from typing import Any, Dict, List, Optional
 import torch
 
 from .. import ops
-from .base import CacheView, Mixer, StateSpec, TensorSpec, register_mixer
+from .base import CacheView, Mixer, ProjectedForm, StateSpec, TensorSpec, register_mixer
 
 
 def _taps(t: torch.Tensor) -> torch.Tensor:
@@ -127,31 +127,33 @@ class Mamba2Mixer(Mixer):
         if not 1 <= n_state <= 256:
             raise ValueError(f"state size {n_state} is outside 1..256")
         self.hidden, self.nh, self.p, self.N, self.G = int(hidden), int(n_heads), int(head_dim), int(n_state), int(groups)
-        self.inner = self.nh * self.p
-        if norm_groups <= 0 or self.inner % norm_groups:
-            raise ValueError(f"{norm_groups} norm groups do not divide {self.inner} channels")
+        self.width = self.nh * self.p
+        if norm_groups <= 0 or self.width % norm_groups:
+            raise ValueError(f"{norm_groups} norm groups do not divide {self.width} channels")
         self.L, self.norm_groups, self.eps, self.sfx = int(conv), int(norm_groups), float(norm_eps), weight_suffix
         self.names = {"in": "in_proj", "conv": "conv1d.weight", "conv_bias": "conv1d.bias", "dt_bias": "dt_bias",
                       "A_log": "A_log", "D": "D", "norm": "norm.weight", "o": "out_proj"}
         if names:
             self.names.update(names)
-        self.channels = self.inner + 2 * self.G * self.N
+        self.channels = self.width + 2 * self.G * self.N
         self.conv_elems = (self.L - 1) * self.channels
         self.w_in = self.w_o = self.taps = self.conv_b = self.A_log = self.dt_bias = self.D = self.norm_w = None
+        #: the norm's weight times a factor on what the out-projection reads
+        self._scaled: Dict[float, torch.Tensor] = {}
 
     def cache_spec(self):
         return StateSpec("mamba2", (self.conv_elems + self.nh * self.N * self.p,), torch.float32)
 
     def tensor_specs(self, prefix: str) -> List[TensorSpec]:
         n, h = self.names, self.hidden
-        return [TensorSpec(f"{prefix}{n['in']}{self.sfx}", (2 * self.inner + 2 * self.G * self.N + self.nh, h)),
+        return [TensorSpec(f"{prefix}{n['in']}{self.sfx}", (2 * self.width + 2 * self.G * self.N + self.nh, h)),
                 TensorSpec(f"{prefix}{n['conv']}", (self.channels, self.L), role="vector"),
                 TensorSpec(f"{prefix}{n['conv_bias']}", (self.channels,), role="vector"),
                 TensorSpec(f"{prefix}{n['dt_bias']}", (self.nh,), role="vector"),
                 TensorSpec(f"{prefix}{n['A_log']}", (self.nh,), role="vector", init="zeros"),
                 TensorSpec(f"{prefix}{n['D']}", (self.nh,), role="vector", init="ones"),
-                TensorSpec(f"{prefix}{n['norm']}", (self.inner,), role="vector", init="ones"),
-                TensorSpec(f"{prefix}{n['o']}{self.sfx}", (h, self.inner))]
+                TensorSpec(f"{prefix}{n['norm']}", (self.width,), role="vector", init="ones"),
+                TensorSpec(f"{prefix}{n['o']}{self.sfx}", (h, self.width))]
 
     def bind(self, tensors, prefix, dtype):
         n = self.names
@@ -163,18 +165,32 @@ class Mamba2Mixer(Mixer):
         self.A_log = tensors[f"{prefix}{n['A_log']}"].contiguous()
         self.D = tensors[f"{prefix}{n['D']}"].contiguous()
         self.norm_w = tensors[f"{prefix}{n['norm']}"].contiguous()
+        self._scaled = {}
 
     def forward(self, a: torch.Tensor, ctx: Any, cache: CacheView) -> torch.Tensor:
-        inner, C = self.inner, self.channels
-        h = ops.linear(a, self.w_in)
+        return ops.linear(self._run(ops.linear(a, self.w_in), 0, ctx, cache), self.w_o)
+
+    def pieces(self):
+        return ProjectedForm(self.w_in, None, self.w_o, None)
+
+    def inner(self, h, at, ctx, cache, out, scale):
+        if scale not in self._scaled:
+            self._scaled[scale] = (self.norm_w * scale).contiguous()
+        self._run(h, at, ctx, cache, out, self._scaled[scale])
+
+    def _run(self, h: torch.Tensor, at: int, ctx: Any, cache: CacheView, out: Optional[torch.Tensor] = None,
+             norm_w: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Everything between the projections on columns ``at ..`` of ``h``."""
+        inner, C = self.width, self.channels
         state = cache.tensor
-        xbc = ops.causal_conv_silu(h[:, inner:inner + C], self.taps, self.conv_b, state, ctx.state_slots, ctx.tok_seq,
+        c0, d0 = at + inner, at + inner + C
+        xbc = ops.causal_conv_silu(h[:, c0:d0], self.taps, self.conv_b, state, ctx.state_slots, ctx.tok_seq,
                                    ctx.cu_q, ctx.positions, ctx.max_q, ctx.status)
-        y = ops.state_space(xbc, h[:, inner + C:inner + C + self.nh], self.A_log, self.dt_bias, self.D, state,
+        y = ops.state_space(xbc, h[:, d0:d0 + self.nh], self.A_log, self.dt_bias, self.D, state,
                             self.conv_elems, ctx.state_slots, ctx.cu_q, ctx.positions, self.nh, self.G, self.N, self.p,
                             ctx.status, max_q=ctx.max_q)
-        out = ops.gated_group_rmsnorm(y, h[:, :inner], self.norm_w, self.eps, inner // self.norm_groups, True, h.dtype)
-        return ops.linear(out, self.w_o)
+        return ops.gated_group_rmsnorm(y, h[:, at:c0], self.norm_w if norm_w is None else norm_w, self.eps,
+                                       inner // self.norm_groups, True, h.dtype, out=out)
 
 
 class RGLRUMixer(Mixer):
