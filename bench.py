@@ -156,7 +156,7 @@ def model_numbers(runner):
     gathers a few rows of it and the tied head reads all of it), and matrix-product parameters."""
     wbytes, mm_params = 0, 0
     for label, t in part_tensors(runner.plan):
-        if label == "TokenEmbedding.table":
+        if label in ("TokenEmbedding.table", "TokenEmbedding.bigram_table"):
             continue                      # (reached only when untied) a table is gathered from, not streamed
         wbytes += t.numel() * t.element_size()
         if t.dim() == 2 and t.shape[0] > 8:
@@ -204,7 +204,8 @@ OPS = {"embed": "elementwise", "add_residual_ss": "elementwise", "resolve_tokens
        "softcap": "hyper", "causal_conv": "recurrent", "rglru": "rglru", "relu_squared": "moe", "moe_route": "moe",
        "moe_experts": "moe", "matrix_memory": "linear_memory", "gated_linear_attention": "linear_memory",
        "scaled_add_rmsnorm": "elementwise", "latent_prepare": "latent", "latent_rotate_q": "latent",
-       "latent_attention": "attention_masked", "moe_table_route": "moe", "head_products": "library"}
+       "latent_attention": "attention_masked", "moe_table_route": "moe", "head_products": "library",
+       "embed_bigram": "elementwise", "shift_add_rmsnorm": "elementwise", "xielu": "elementwise"}
 
 
 class OpLog:
@@ -835,9 +836,37 @@ def nelosun_sizes(name):
     return ne, rapolix_sizes(name)[0], demazen_sizes(name)[0]
 
 
+def givavik_sizes(name):
+    """Givavik layers at the widths of LFM2-<name>: latent attention with as many heads as the LFM2 stack, of 64 + 32
+    (values of 64), over a cached row of 256 + 32, every second such layer reading the latents of the one before it;
+    attention with the same heads as the LFM2 stack (keys and values of 64, sigmoid weights, a cap of 50) beside Mamba-2
+    with twice the width inside (heads of 64, state 128); a dense feed-forward of the LFM2 stack's width with xIELU beside
+    every mixer; a bigram table; eight layers.  Beside it Nelosun (latent attention, attention on the same kernels with a
+    softmax, the same arrangement of a layer) and Vukavik (Mamba-2, attention, dense feed-forwards) at the same widths."""
+    from vapi_b200.models.lfm2 import Lfm2Config
+    lf = lfm2_sizes(name)
+    W, ff = lf["hidden_size"], Lfm2Config.effective_ff_dim(lf)
+    heads = lf["num_attention_heads"]
+    mlp = {"kind": "dense", "ff": ff}
+
+    def lat(source=None):
+        m = {"heads": heads, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 256, "scale": 0.1, "rot": {"base": 1000000.0, "dims": 32}}
+        return {"type": "latent_attention", "mlp": mlp, "mixer": m if source is None else dict(m, kv_from=source)}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": heads, "kv_heads": lf["num_key_value_heads"], "dim": 64, "vdim": 64, "scale": 0.125, "softcap": 50.0,
+                 "rot": {"base": 500000.0, "dims": 32}},
+        "right": {"heads": 2 * W // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1},
+        "left_scale": 1.2, "right_scale": 1.1}}
+    gv = {"architecture": "Givavik", "vocab": lf["vocab_size"], "width": W, "norm": {"eps": 1e-5},
+          "embedding": {"scale": 1.0, "bigram": {"buckets": 16381, "mul_prev": 31337, "mul_cur": 911}},
+          "layers": [lat(), par, lat(0), par, lat(), par, lat(4), par]}
+    return gv, nelosun_sizes(name)[0], vukavik_sizes(name)[0]
+
+
 def mixers(args):
     """``--only mixers``: prefill and decode of eight layers of ``--design`` beside LFM2 layers (Vukavik, Rapolix; Demazen
-    stands beside Vukavik and Rapolix, whose kernels are the nearest to its own, Nelosun beside Rapolix and Demazen)
+    stands beside Vukavik and Rapolix, whose kernels are the nearest to its own, Nelosun beside Rapolix and Demazen, Givavik
+    beside Nelosun and Vukavik)
     of equal width (random weights), and where each model's time goes, kernel family by kernel family."""
     import torch
     from vapi_b200 import ops
@@ -858,6 +887,9 @@ def mixers(args):
     elif args.design == "nelosun":
         ne, rp, dz = nelosun_sizes(args.sizes)
         models = (("nelosun", ne), ("rapolix", rp), ("demazen", dz))
+    elif args.design == "givavik":
+        gv, ne, vk = givavik_sizes(args.sizes)
+        models = (("givavik", gv), ("nelosun", ne), ("vukavik", vk))
     else:
         vk, lf = rapolix_sizes(args.sizes) if args.design == "rapolix" else vukavik_sizes(args.sizes)
         models = ((args.design, vk), ("lfm2", lf))
@@ -1029,9 +1061,9 @@ def main():
                          "and print what one step's kernels did inside the captured graph, or (mixers) prefill and "
                          "decode of eight Vukavik layers beside eight LFM2 layers of equal width, kernel family by kernel family")
     ap.add_argument("--sizes", default="1.2b", choices=["1.2b", "700m", "2.6b"], help="layer sizes of LFM2-<sizes>")
-    ap.add_argument("--design", default="vukavik", choices=["vukavik", "rapolix", "demazen", "nelosun"],
+    ap.add_argument("--design", default="vukavik", choices=["vukavik", "rapolix", "demazen", "nelosun", "givavik"],
                     help="with --only mixers: the architecture whose layers stand beside LFM2's (demazen: beside Vukavik's and "
-                         "Rapolix's; nelosun: beside Rapolix's and Demazen's)")
+                         "Rapolix's; nelosun: beside Rapolix's and Demazen's; givavik: beside Nelosun's and Vukavik's)")
     ap.add_argument("--page-size", type=int, default=0, help="tokens per cache page (0: the engine's default)")
     ap.add_argument("--dtype", default="bfloat16", help="bfloat16 (serving) or float32 (the true 32-bit path)")
     ap.add_argument("--no-fp32", action="store_true", help="leave the float32 points out of the default run")

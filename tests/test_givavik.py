@@ -549,7 +549,17 @@ def test_joined_projections_are_the_branches_with_their_factors(device, dtype, f
     mixer = r.plan.layers[layer_at].mixer
     a = torch.randn((n, r.plan.hidden_size), generator=torch.Generator().manual_seed(1)).to(device)
     joint = mixer.forward(a, ctx, view)
-    alone = sum(f * m.forward(a, ctx, v) for m, f, v in zip(mixer.branches, mixer.factors, view.parts))
+    assert mixer.branches[0].w_qkv is None and mixer.branches[1].w_o is None, "nobody keeps the projections twice"
+    from vapi_b200.config.model import load_config_json, resolve_architecture
+    from vapi_b200.weights.loader import load_tensors
+    cfg = load_config_json(folders[name])
+    arch = resolve_architecture(cfg)
+    again = arch.plan(arch.parse(cfg))
+    tensors = load_tensors(folders[name], again.tensor_specs(), dtype, device)
+    alone = torch.zeros_like(a)
+    for sub, m, f, v in zip(("left.", "right."), again.layers[layer_at].mixer.branches, mixer.factors, view.parts):
+        m.bind(tensors, f"l{layer_at}.mix." + sub, dtype)
+        alone += f * m.forward(a, ctx, v)
     _close(joint, alone, 1e-5)
     from vapi_b200.parts import GQAttention, ParallelMixer, ShortConv
     with pytest.raises(ValueError):

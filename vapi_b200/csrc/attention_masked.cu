@@ -267,16 +267,22 @@ masked_attention_kernel(const T* __restrict__ q, long long q_row_stride, const T
     }
 }
 
-// Partial results of `splits` (at most 32) blocks combined in split order: one warp per (token, head).
+// Partial results of `splits` (at most 32) blocks combined in split order: a warp takes 64 columns of one (token, head),
+// a lane two of them, so that a decode step's few rows still make enough warps.
+constexpr int MC_COLS = 64;
 template <typename T>
-__global__ void masked_attention_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                                const T* __restrict__ gate, long long gate_stride, T* __restrict__ out,
-                                                long long rows, int nh, int dv, int splits, const ScoreForm form) {
-    const long long row = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+__global__ void __launch_bounds__(128)
+masked_attention_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                const T* __restrict__ gate, long long gate_stride, T* __restrict__ out,
+                                long long rows, int nh, int dv, int splits, const ScoreForm form) {
+    const int chunks = (dv + MC_COLS - 1) / MC_COLS;
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     pdl_trigger();
     pdl_wait();
+    const long long row = item / chunks;
     if (row >= rows) return;
+    const int col = (int)(item - row * chunks) * MC_COLS + 2 * lane;
     float ms = -INFINITY, ls = 0.f;
     if (lane < splits) {
         ms = part_ml[(row * splits + lane) * 2];
@@ -285,25 +291,30 @@ __global__ void masked_attention_combine_kernel(const float* __restrict__ part_o
     const float mx = warp_max(ms);
     // weights that are not normalised over the keys simply add up
     const float w = form.sigmoid ? 1.f : (ms == -INFINITY ? 0.f : expf(ms - mx));
-    float lsum = 0.f;
-    for (int sp = 0; sp < splits; ++sp) lsum += __shfl_sync(0xffffffffu, ls * w, sp);
+    const float* po = part_o + row * splits * (size_t)dv + col;
+    const bool mine = col < dv;                                     // (widths are multiples of 4: a lane has two columns or none)
+    float lsum = 0.f, o0 = 0.f, o1 = 0.f;
+#pragma unroll 4
+    for (int sp = 0; sp < splits; ++sp) {
+        const float2 v = mine ? *reinterpret_cast<const float2*>(po + (size_t)sp * dv) : make_float2(0.f, 0.f);
+        const float ws = __shfl_sync(0xffffffffu, w, sp);
+        lsum += __shfl_sync(0xffffffffu, ls * w, sp);
+        o0 = fmaf(v.x, ws, o0);
+        o1 = fmaf(v.y, ws, o1);
+    }
     float inv = form.sigmoid ? 1.f : (lsum > 0.f ? 1.f / lsum : 0.f);
     const long long tok = row / nh;
     const int h = (int)(row - tok * nh);
     inv *= form.out_scale;
-    if (gate) {
-        inv *= 1.f / (1.f + expf(-to_f32(gate[(size_t)tok * gate_stride + h])));
+    if (gate) inv *= 1.f / (1.f + expf(-to_f32(gate[(size_t)tok * gate_stride + h])));
+    if (mine) {
+        T* dst = out + (size_t)tok * form.out_stride + (size_t)h * dv + col;
+        dst[0] = from_f32<T>(o0 * inv);
+        dst[1] = from_f32<T>(o1 * inv);
     }
-    for (int c0 = 0; c0 < dv; c0 += 32) {
-        const int col = c0 + lane;
-        float o = 0.f;
-        for (int sp = 0; sp < splits; ++sp) {
-            const float ws = __shfl_sync(0xffffffffu, w, sp);
-            const float v = col < dv ? part_o[(row * splits + sp) * (size_t)dv + col] : 0.f;
-            o += v * ws;
-        }
-        if (col < dv) out[(size_t)tok * form.out_stride + (size_t)h * dv + col] = from_f32<T>(o * inv);
-    }
+}
+static int combine_blocks(long long rows, int dv) {
+    return (int)((rows * ((dv + MC_COLS - 1) / MC_COLS) + 3) / 4);
 }
 
 template <typename T, int DVMAX>
@@ -332,7 +343,7 @@ static int launch_masked(const void* q, long long q_row_stride, const void* cach
     int rc = check_launch("masked_attention", e);
     if (rc != 0 || splits == 1) return rc;
     const long long rows = (long long)n * nh;
-    e = launch(masked_attention_combine_kernel<T>, (int)((rows + 3) / 4), 128, 0, stream, (const float*)part_o,
+    e = launch(masked_attention_combine_kernel<T>, combine_blocks(rows, dv), 128, 0, stream, (const float*)part_o,
                (const float*)part_ml, (const T*)gate, gate_stride, (T*)out, rows, nh, dv, splits, form);
     return check_launch("masked_attention_combine", e);
 }
@@ -399,7 +410,7 @@ VAPI_EXPORT int vapi_masked_attention(const void* q, long long q_row_stride, con
         if (rc != 0 || splits == 1) return rc;
         const long long rows = (long long)n * nh;
         return check_launch("masked_attention_combine",
-                            launch(masked_attention_combine_kernel<__nv_bfloat16>, (int)((rows + 3) / 4), 128, 0, stream,
+                            launch(masked_attention_combine_kernel<__nv_bfloat16>, combine_blocks(rows, dv), 128, 0, stream,
                                    (const float*)part_o, (const float*)part_ml, (const __nv_bfloat16*)gate, gate_stride,
                                    (__nv_bfloat16*)out, rows, nh, dv, splits, form));
     }
@@ -411,7 +422,7 @@ VAPI_EXPORT int vapi_masked_attention(const void* q, long long q_row_stride, con
         if (rc != 0 || splits == 1) return rc;
         const long long rows = (long long)n * nh;
         return check_launch("masked_attention_combine",
-                            launch(masked_attention_combine_kernel<__nv_bfloat16>, (int)((rows + 3) / 4), 128, 0, stream,
+                            launch(masked_attention_combine_kernel<__nv_bfloat16>, combine_blocks(rows, dv), 128, 0, stream,
                                    (const float*)part_o, (const float*)part_ml, (const __nv_bfloat16*)nullptr, (long long)0,
                                    (__nv_bfloat16*)out, rows, nh, dv, splits, form));
     }

@@ -66,8 +66,9 @@ struct ScoreForm {
 // The sigmoid form with its constants worked out for base-2 exponentials: with a raw product s = q.k,
 //   capped:  weight = 1 / (1 + 2^(kc * tanh(k1 * s) + nb)),  k1 = scale / cap, kc = -cap * log2 e
 //   else     weight = 1 / (1 + 2^(k1 * s + nb)),             k1 = -scale * log2 e
-// and nb = -bias[head] * log2 e, a row's own number.
-struct SigmoidForm { float k1 = 0.f, kc = 0.f; int capped = 0; };
+// and nb = -bias[head] * log2 e, a row's own number.  near: the |s| below which kc * tanh(k1 * s) is taken from tanh's
+// odd Taylor polynomial, whose coefficients p[] are already those of s.
+struct SigmoidForm { float k1 = 0.f, kc = 0.f, near = 0.f; float p[4] = {0.f, 0.f, 0.f, 0.f}; int capped = 0; };
 
 inline SigmoidForm sigmoid_form(float scale, float softcap) {
     SigmoidForm f;
@@ -75,6 +76,12 @@ inline SigmoidForm sigmoid_form(float scale, float softcap) {
     f.capped = softcap > 0.f;
     f.k1 = f.capped ? scale / softcap : -scale * log2e;
     f.kc = f.capped ? -softcap * log2e : 0.f;
+    if (f.capped && scale != 0.f) {
+        const double k = f.k1, taylor[4] = {1.0, -1.0 / 3.0, 2.0 / 15.0, -17.0 / 315.0};
+        double power = k;
+        for (int i = 0; i < 4; ++i, power *= k * k) f.p[i] = (float)(f.kc * taylor[i] * power);
+        f.near = 0.2f / (f.k1 < 0.f ? -f.k1 : f.k1);
+    }
     return f;
 }
 
@@ -90,30 +97,26 @@ __device__ __forceinline__ float rcp_ftz(float x) {
 }
 
 // N raw products of one row -> their weights, in place.  Every lane of the warp must take part.  The products of normed
-// queries and keys usually stay far below the cap, so tanh is its odd Taylor polynomial while no lane's |k1 s| reaches
-// 0.3 (error below 2e-8) and 1 - 2 / (1 + e^2u) otherwise; two weights share one reciprocal, 1/a = b / (ab) (exponents
-// are clamped at 62, where a weight is below 2^-61, so that the product stays finite).
+// queries and keys usually stay far below the cap, so tanh is its Taylor polynomial while no lane's |k1 s| reaches 0.2
+// (relative error below 6e-8) and 1 - 2 / (1 + e^2u) otherwise; two weights share one reciprocal, 1/a = b / (ab)
+// (exponents are clamped at 62, where a weight is below 2^-61, so that the product stays finite).
 template <int N>
 __device__ __forceinline__ void sigmoid_weights(float (&s)[N], const SigmoidForm& f, float nb) {
     static_assert(N % 2 == 0, "weights come in pairs");
     if (f.capped) {
-        float um = 0.f;
+        float sm = 0.f;
 #pragma unroll
-        for (int i = 0; i < N; ++i) {
-            s[i] *= f.k1;
-            um = fmaxf(um, fabsf(s[i]));
-        }
-        if (!__any_sync(0xffffffffu, um >= 0.3f)) {
+        for (int i = 0; i < N; ++i) sm = fmaxf(sm, fabsf(s[i]));
+        if (!__any_sync(0xffffffffu, !(sm < f.near))) {
 #pragma unroll
             for (int i = 0; i < N; ++i) {
-                const float u = s[i], z = u * u;
-                const float t = fmaf(z, fmaf(z, fmaf(z, fmaf(z, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
-                s[i] = fmaf(u * t, f.kc, nb);
+                const float z = s[i] * s[i];
+                s[i] = fmaf(s[i], fmaf(z, fmaf(z, fmaf(z, f.p[3], f.p[2]), f.p[1]), f.p[0]), nb);
             }
         } else {
 #pragma unroll
             for (int i = 0; i < N; ++i) {
-                const float e = ex2_ftz(fminf(s[i] * 2.8853900817779268f, 126.f));
+                const float e = ex2_ftz(fminf(s[i] * (f.k1 * 2.8853900817779268f), 126.f));
                 s[i] = fmaf(fmaf(-2.f, rcp_ftz(1.f + e), 1.f), f.kc, nb);
             }
         }

@@ -451,9 +451,8 @@ struct ShiftIndex {
     float* state; long long slot_stride; int num_slots; int* status;
 };
 
-constexpr int SHIFT_KMAX = 4;
-
-template <typename T>
+// SHIFT_KMAX: 16-byte pieces of a row in a thread's registers
+template <typename T, int SHIFT_KMAX>
 __global__ void __launch_bounds__(256)
 shift_add_rmsnorm_vec_kernel(const float* __restrict__ x, const T* __restrict__ y1, const float* __restrict__ s1,
                              const T* __restrict__ y2, const float* __restrict__ s2, const float* __restrict__ w, float eps,
@@ -622,18 +621,22 @@ VAPI_EXPORT int vapi_shift_add_rmsnorm(const float* x, const void* y1, const flo
                            (uintptr_t)state) & 15) == 0 && slot_stride % 4 == 0 &&
                          (((uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)out_h | (uintptr_t)out_s) & (4 * esz - 1)) == 0;
     const int vt = hidden > 1024 ? 256 : 128;
-    const bool vec = hidden % 4 == 0 && hidden / 4 <= SHIFT_KMAX * vt && aligned;
+    const int pieces = (hidden / 4 + vt - 1) / vt;
+    const bool vec = hidden % 4 == 0 && pieces <= 4 && aligned;
     const int rpb = rows_per_block > 0 ? rows_per_block : 1;
     cudaError_t e;
+#define SHIFT_VEC(T, K)                                                                                                          \
+    launch(shift_add_rmsnorm_vec_kernel<T, K>, (n + rpb - 1) / rpb, vt, 0, stream, x, (const T*)y1, s1, (const T*)y2, s2, w, eps, \
+           shift, ix, x_out, (T*)out_h, (T*)out_s, n, hidden, rpb)
 #define SHIFT_GO(T)                                                                                                            \
-    e = vec ? launch(shift_add_rmsnorm_vec_kernel<T>, (n + rpb - 1) / rpb, vt, 0, stream, x, (const T*)y1, s1, (const T*)y2,   \
-                     s2, w, eps, shift, ix, x_out, (T*)out_h, (T*)out_s, n, hidden, rpb)                                       \
-            : launch(shift_add_rmsnorm_kernel<T>, n, 256, 0, stream, x, (const T*)y1, s1, (const T*)y2, s2, w, eps, shift, ix, \
-                     x_out, (T*)out_h, (T*)out_s, n, hidden)
+    e = !vec ? launch(shift_add_rmsnorm_kernel<T>, n, 256, 0, stream, x, (const T*)y1, s1, (const T*)y2, s2, w, eps, shift,    \
+                      ix, x_out, (T*)out_h, (T*)out_s, n, hidden)                                                              \
+             : pieces <= 1 ? SHIFT_VEC(T, 1) : pieces <= 2 ? SHIFT_VEC(T, 2) : SHIFT_VEC(T, 4)
     if (dtype == VAPI_F32) SHIFT_GO(float);
     else if (dtype == VAPI_BF16) SHIFT_GO(__nv_bfloat16);
     else return fail(-2, "shift_add_rmsnorm: unsupported dtype %d", dtype);
 #undef SHIFT_GO
+#undef SHIFT_VEC
     return check_launch("shift_add_rmsnorm", e);
 }
 
@@ -1008,6 +1011,9 @@ VAPI_EXPORT int vapi_postnorm_add_rmsnorm(float* x, const void* y, int dtype, co
 
 // xIELU elementwise (where it does not ride on a product): out = xielu(z), consts = {up, down}; four elements a
 // thread with 8- / 16-byte accesses, the last few one by one.
+__device__ __forceinline__ float xielu_as(float, float z, float up, float down) { return xielu(z, up, down); }
+__device__ __forceinline__ float xielu_as(__nv_bfloat16, float z, float up, float down) { return xielu_16(z, up, down); }
+
 template <typename T>
 __global__ void xielu_kernel(const T* __restrict__ z, T* __restrict__ out, const float* __restrict__ consts, size_t total, int vec) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -1017,9 +1023,10 @@ __global__ void xielu_kernel(const T* __restrict__ z, T* __restrict__ out, const
     const size_t i0 = i * 4;
     if (vec && i0 + 3 < total) {
         const float4 v = Pack4<T>::load(z + i0);
-        Pack4<T>::store(out + i0, make_float4(xielu(v.x, up, down), xielu(v.y, up, down), xielu(v.z, up, down), xielu(v.w, up, down)));
+        Pack4<T>::store(out + i0, make_float4(xielu_as(T(), v.x, up, down), xielu_as(T(), v.y, up, down),
+                                             xielu_as(T(), v.z, up, down), xielu_as(T(), v.w, up, down)));
     } else {
-        for (size_t j = i0; j < i0 + 4 && j < total; ++j) out[j] = from_f32<T>(xielu(to_f32(z[j]), up, down));
+        for (size_t j = i0; j < i0 + 4 && j < total; ++j) out[j] = from_f32<T>(xielu_as(T(), to_f32(z[j]), up, down));
     }
 }
 
@@ -1121,6 +1128,50 @@ __global__ void gated_group_rmsnorm_wide_kernel(const float* __restrict__ y, con
     }
 }
 
+// Wide groups with 16-byte accesses, each value read once and kept in registers: two pieces of four columns a thread.
+template <typename T>
+__global__ void __launch_bounds__(1024)
+gated_group_rmsnorm_vec_kernel(const float* __restrict__ y, const T* __restrict__ z, long long z_stride,
+                               const float* __restrict__ w, int w_len, float eps, int gate_first, T* __restrict__ out, int n,
+                               int width, int group, long long out_stride) {
+    __shared__ float red[33];
+    const int groups = width / group;
+    const int t = blockIdx.x / groups, g = blockIdx.x - t * groups;
+    const int sig = gate_first & 2;
+    gate_first &= 1;
+    pdl_trigger();
+    pdl_wait();
+    const float* yr = y + (size_t)t * width + (size_t)g * group;
+    const T* zr = z + (size_t)t * z_stride + (size_t)g * group;
+    float4 v[2], gt[2];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int c = 4 * (threadIdx.x + k * blockDim.x);
+        v[k] = gt[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < group) {
+            v[k] = Pack4<float>::load(yr + c);
+            const float4 zv = Pack4<T>::load(zr + c);
+            gt[k] = make_float4(norm_gate(zv.x, sig), norm_gate(zv.y, sig), norm_gate(zv.z, sig), norm_gate(zv.w, sig));
+            if (gate_first) { v[k].x *= gt[k].x; v[k].y *= gt[k].y; v[k].z *= gt[k].z; v[k].w *= gt[k].w; }
+            ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+        }
+    }
+    ss = block_sum(ss, red);
+    const float inv = rsqrtf(ss / (float)group + eps);
+    T* orow = out + (size_t)t * out_stride + (size_t)g * group;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int c = 4 * (threadIdx.x + k * blockDim.x);
+        if (c < group) {
+            const float4 wv = Pack4<float>::load(w + (g * group + c) % w_len);
+            float4 o = make_float4(v[k].x * inv * wv.x, v[k].y * inv * wv.y, v[k].z * inv * wv.z, v[k].w * inv * wv.w);
+            if (!gate_first) { o.x *= gt[k].x; o.y *= gt[k].y; o.z *= gt[k].z; o.w *= gt[k].w; }
+            Pack4<T>::store(orow + c, o);
+        }
+    }
+}
+
 VAPI_EXPORT int vapi_gated_group_rmsnorm(const float* y, const void* z, long long z_stride, int dtype, const float* w,
                                          int w_len, float eps, int gate_first, void* out, int n, int width, int group,
                                          cudaStream_t stream, long long out_stride) {
@@ -1132,6 +1183,19 @@ VAPI_EXPORT int vapi_gated_group_rmsnorm(const float* y, const void* z, long lon
     const int warps = 4;
     const int blocks = (int)((items + warps - 1) / warps);
     cudaError_t e;
+    const int esz = dtype == VAPI_F32 ? 4 : 2;
+    const bool vec = group >= 512 && group <= 8192 && group % 4 == 0 && w_len % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0 &&
+                     (((uintptr_t)y | (uintptr_t)w) & 15) == 0 && (((uintptr_t)z | (uintptr_t)out) & (4 * esz - 1)) == 0;
+    if (vec && items <= 0x7fffffffLL && (dtype == VAPI_F32 || dtype == VAPI_BF16)) {
+        const int threads = ((group / 8 + 31) / 32) * 32;
+        if (dtype == VAPI_F32)
+            e = launch(gated_group_rmsnorm_vec_kernel<float>, (int)items, threads, 0, stream, y, (const float*)z, z_stride, w, w_len,
+                       eps, gate_first, (float*)out, n, width, group, out_stride);
+        else
+            e = launch(gated_group_rmsnorm_vec_kernel<__nv_bfloat16>, (int)items, threads, 0, stream, y, (const __nv_bfloat16*)z,
+                       z_stride, w, w_len, eps, gate_first, (__nv_bfloat16*)out, n, width, group, out_stride);
+        return check_launch("gated_group_rmsnorm", e);
+    }
     if (group >= 512 && items <= 0x7fffffffLL && (dtype == VAPI_F32 || dtype == VAPI_BF16)) {
         const int threads = group >= 2048 ? 256 : 128;
         if (dtype == VAPI_F32)

@@ -263,7 +263,7 @@ __device__ __forceinline__ void gv_tile_finish(const GvParams& p, int tile, int 
         const bool valid = i < R && n < p.N && m < p.M;
         if (valid && p.bias) y += p.bias[n];
         if (EPI == GV_EPI_BF16) {
-            if (p.xielu) y = xielu(y, p.xielu[0], p.xielu[1]);
+            if (p.xielu) y = xielu_16(y, p.xielu[0], p.xielu[1]);
             if (valid) p.out_bf16[(size_t)m * p.out_stride + n] = __float2bfloat16_rn(y);
         } else if (EPI == GV_EPI_F32) {
             if (valid) p.out_f32[(size_t)m * p.out_stride + n] = y;

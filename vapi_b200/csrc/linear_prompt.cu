@@ -369,7 +369,7 @@ prompt_linear_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
                     if (p.xielu) {
                         const float up = p.xielu[0], down = p.xielu[1];
 #pragma unroll
-                        for (int j = 0; j < 32; ++j) v[j] = xielu(v[j], up, down);
+                        for (int j = 0; j < 32; ++j) v[j] = xielu_16(v[j], up, down);
                     }
                     if (fast) {
                         put(v);

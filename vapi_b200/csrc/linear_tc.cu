@@ -205,7 +205,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant
             if (p.xielu) {
                 const float up = p.xielu[0], down = p.xielu[1];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) vv[i] = xielu(vv[i], up, down);
+                for (int i = 0; i < 4; ++i) vv[i] = xielu_16(vv[i], up, down);
             }
             __nv_bfloat16* o = p.out_bf16 + (size_t)m * p.out_stride + f0;
             if (full && (p.out_stride & 3) == 0) {

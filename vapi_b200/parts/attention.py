@@ -179,6 +179,9 @@ class GQAttention(Mixer):
             return None
         return ProjectedForm(self.w_qkv, self.b_qkv, self.w_o, self.b_o, first=True)
 
+    def give_up_projections(self):
+        self.w_qkv = self.b_qkv = self.w_o = self.b_o = None
+
     def inner(self, h, at, ctx, cache, out, scale):
         if at != 0:
             raise ValueError("q, k and v lead the rows of their product")

@@ -289,6 +289,11 @@ class Mixer(Part):
         """This (bound) mixer's projections, or None if it is not of that form."""
         return None
 
+    def give_up_projections(self) -> None:
+        """Whoever joined the projections holds them now: drop this mixer's own copies (it then runs only through
+        :meth:`inner`)."""
+        raise NotImplementedError
+
     def inner(self, h: torch.Tensor, at: int, ctx: "Any", cache: CacheView, out: torch.Tensor, scale: float) -> None:
         """What lies between the projections: reads columns ``at ..`` of ``h`` [n, columns], writes ``scale`` times the
         out-projection's input into ``out`` [n, its width] (unit inner stride, rows of a wider buffer)."""

@@ -7,7 +7,7 @@ from typing import Any, Dict, List, Optional, Sequence, Tuple
 import torch
 
 from .. import ops
-from .base import CacheView, Mixer, ProjectedForm, TensorSpec, register_mixer
+from .base import CacheView, Mixer, TensorSpec, register_mixer
 
 
 @dataclass
@@ -48,7 +48,7 @@ class ParallelMixer(Mixer):
         if self.factors is not None and (len(self.factors) != len(branches) or deferred):
             raise ValueError("one factor per branch, and no norms to defer")
         self.deferred = bool(deferred) and len(branches) <= 2
-        self._pieces: Optional[List[ProjectedForm]] = None
+        self._joined = False
         self.w_in = self.b_in = self.w_out = self.b_out = None
         self.subs = [s for s, _ in branches]
         self.branches: List[Mixer] = [m for _, m in branches]
@@ -120,7 +120,9 @@ class ParallelMixer(Mixer):
             for p, f in zip(pieces, self.factors):
                 if p.b_out is not None:
                     self.b_out += f * p.b_out
-        self._pieces = pieces
+        self._joined = True
+        for m in self.branches:
+            m.give_up_projections()
 
     def _forward_joined(self, a: torch.Tensor, ctx: Any, views) -> torch.Tensor:
         h = ops.linear(a, self.w_in, self.b_in)
@@ -136,7 +138,7 @@ class ParallelMixer(Mixer):
 
     def forward(self, a: torch.Tensor, ctx: Any, cache: CacheView) -> torch.Tensor:
         views = cache.parts if cache.kind == "multi" else [cache] * len(self.branches)
-        if self._pieces is not None:
+        if self._joined:
             return self._forward_joined(a, ctx, views)
         outs = [m.forward(a, ctx, v) for m, v in zip(self.branches, views)]
         if self.deferred:

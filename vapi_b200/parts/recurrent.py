@@ -173,6 +173,9 @@ class Mamba2Mixer(Mixer):
     def pieces(self):
         return ProjectedForm(self.w_in, None, self.w_o, None)
 
+    def give_up_projections(self):
+        self.w_in = self.w_o = None
+
     def inner(self, h, at, ctx, cache, out, scale):
         if scale not in self._scaled:
             self._scaled[scale] = (self.norm_w * scale).contiguous()
