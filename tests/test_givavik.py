@@ -340,7 +340,7 @@ def test_bigram_rows_and_the_token_they_carry(dtype):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_xielu_alone_and_behind_a_product(dtype):
     """Elementwise at sizes that are no multiple of four, values from far below zero to far above, both sides of zero;
-    then as the epilogue of every product that takes it (1 to 16, 17 to 32 and 256 rows and more) and behind the library's."""
+    then as the epilogue of every product that takes it (1 to 16, 17 to 32 and prompt-sized steps) and behind the library's."""
     from vapi_b200 import ops
     g = torch.Generator().manual_seed(7)
     consts = torch.tensor([0.83, 1.21])
@@ -349,12 +349,14 @@ def test_xielu_alone_and_behind_a_product(dtype):
     near = z[-5:].float()
     got = ops.xielu(near.cuda(), consts.cuda()).cpu()
     assert torch.allclose(got, plain_ops.xielu(near.double(), consts.double()).float(), rtol=1e-4, atol=1e-9), "digits are kept next to zero"
-    for n, K, N in ((1, 64, 40), (7, 96, 136), (16, 320, 72), (20, 64, 200), (32, 192, 136), (100, 64, 96), (256, 128, 200), (300, 72, 264)):
+    for n, K, N in ((1, 64, 40), (7, 96, 136), (16, 320, 72), (20, 64, 200), (32, 192, 136), (100, 64, 96), (256, 128, 200), (300, 72, 264), (1030, 64, 72)):
         x, w = (torch.randn((n, K), generator=g)).to(dtype), (torch.randn((N, K), generator=g) * 0.2).to(dtype)
         want = plain_ops.xielu(x.float() @ w.float().t(), consts)
         got = ops.linear_xielu(x.cuda(), w.cuda(), consts.cuda())
         assert got.dtype == dtype and got.shape == (n, N)
         _close(got, want, 2e-5 if dtype == torch.float32 else 2e-2)
+        if dtype == torch.bfloat16 and n > 32:
+            _close(ops.prompt_linear(w.cuda(), act=x.cuda(), epilogue="bf16", xielu=consts.cuda()), want, 2e-2)
 
 
 @pytest.mark.gpu
