@@ -25,7 +25,7 @@ def left(heads=4, kv_heads=2, dim=16, vdim=24, scale=0.3, softcap: Optional[floa
     return m
 
 
-def right(heads=6, vdim=12, state=20, groups=3, conv=3, norm_groups=2) -> dict:
+def right(heads=6, vdim=10, state=20, groups=3, conv=3, norm_groups=2) -> dict:
     return {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": norm_groups}
 
 

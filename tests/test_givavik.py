@@ -69,8 +69,8 @@ def test_the_architecture_is_found_by_its_name_and_every_size_comes_from_the_con
     assert shapes["l0.mix.left.q"] == (64, 64) and shapes["l0.mix.left.k"] == (32, 64) and shapes["l0.mix.left.v"] == (48, 64)
     assert shapes["l0.mix.left.q.b"] == (64,) and shapes["l0.mix.left.o"] == (64, 96) and shapes["l0.mix.left.o.b"] == (64,)
     assert shapes["l0.mix.left.pb"] == (4,) and shapes["l0.shift"] == (64,) and shapes["l0.ls2"] == (64,)
-    assert shapes["l0.mix.right.in"] == (2 * 72 + 2 * 3 * 20 + 6, 64) and shapes["l0.mix.right.conv"] == (72 + 120, 3)
-    assert shapes["l0.mix.right.o"] == (64, 72) and shapes["l0.mlp.up"] == (72, 64) and shapes["l0.mlp.act"] == (2,)
+    assert shapes["l0.mix.right.in"] == (2 * 60 + 2 * 3 * 20 + 6, 64) and shapes["l0.mix.right.conv"] == (60 + 120, 3)
+    assert shapes["l0.mix.right.o"] == (64, 60) and shapes["l0.mlp.up"] == (72, 64) and shapes["l0.mlp.act"] == (2,)
     assert shapes["l1.mix.q"] == (3 * 20, 64) and shapes["l1.mix.dkv"] == (32, 64) and shapes["l1.mix.dkv.norm"] == (24,)
     assert shapes["l1.mix.uk"] == (36, 24) and shapes["l1.mix.uv"] == (60, 24) and shapes["l1.mix.sink"] == (3,) and shapes["l1.mix.o"] == (64, 60)
     assert shapes["l2.mix.q"] == (2 * 28, 64) and shapes["l2.mix.uk"] == (40, 24) and "l2.mix.dkv" not in shapes and "l2.mix.dkv.norm" not in shapes
@@ -96,7 +96,7 @@ def test_the_architecture_is_found_by_its_name_and_every_size_comes_from_the_con
                 [gu.layer(gu.parallel(gu.left(dims=18)))],
                 [gu.layer(gu.parallel(gu.left(softcap=-1.0)))],
                 [gu.layer(gu.parallel(None, gu.right(heads=5, groups=2)))],
-                [gu.layer(gu.parallel(None, gu.right(norm_groups=5)))],
+                [gu.layer(gu.parallel(None, gu.right(norm_groups=7)))],
                 [gu.layer(gu.latent(kv_from=0))],                                               # itself
                 [lat, gu.layer(gu.latent(kv_from=0)), gu.layer(gu.latent(kv_from=1))],          # a layer without a latent of its own
                 [lat, gu.layer(gu.latent(kv_from=0, kv_rank=28))], [lat, gu.layer(gu.latent(kv_from=0, base=7.0))],
