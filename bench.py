@@ -839,7 +839,7 @@ def nelosun_sizes(name):
 def givavik_sizes(name):
     """Givavik layers at the widths of LFM2-<name>: latent attention with as many heads as the LFM2 stack, of 64 + 32
     (values of 64), over a cached row of 256 + 32, every second such layer reading the latents of the one before it;
-    attention with the same heads as the LFM2 stack (keys and values of 64, sigmoid weights, a cap of 50) beside Mamba-2
+    attention with the same heads as the LFM2 stack (keys and values of 64, sigmoid weights, a cap of 40) beside Mamba-2
     with twice the width inside (heads of 64, state 128); a dense feed-forward of the LFM2 stack's width with xIELU beside
     every mixer; a bigram table; eight layers.  Beside it Nelosun (latent attention, attention on the same kernels with a
     softmax, the same arrangement of a layer) and Vukavik (Mamba-2, attention, dense feed-forwards) at the same widths."""
@@ -850,13 +850,13 @@ def givavik_sizes(name):
     mlp = {"kind": "dense", "ff": ff}
 
     def lat(source=None):
-        m = {"heads": heads, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 256, "scale": 0.1, "rot": {"base": 1000000.0, "dims": 32}}
+        m = {"heads": heads, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 256, "scale": 0.1, "rot": {"base": 10000.0, "dims": 32}}
         return {"type": "latent_attention", "mlp": mlp, "mixer": m if source is None else dict(m, kv_from=source)}
     par = {"type": "parallel", "mlp": mlp, "mixer": {
-        "left": {"heads": heads, "kv_heads": lf["num_key_value_heads"], "dim": 64, "vdim": 64, "scale": 0.125, "softcap": 50.0,
-                 "rot": {"base": 500000.0, "dims": 32}},
+        "left": {"heads": heads, "kv_heads": lf["num_key_value_heads"], "dim": 64, "vdim": 64, "scale": 0.125, "softcap": 40.0,
+                 "rot": {"base": 10000.0, "dims": 64}},
         "right": {"heads": 2 * W // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1},
-        "left_scale": 1.2, "right_scale": 1.1}}
+        "left_scale": 0.8, "right_scale": 1.25}}
     gv = {"architecture": "Givavik", "vocab": lf["vocab_size"], "width": W, "norm": {"eps": 1e-5},
           "embedding": {"scale": 1.0, "bigram": {"buckets": 16381, "mul_prev": 31337, "mul_cur": 911}},
           "layers": [lat(), par, lat(0), par, lat(), par, lat(4), par]}

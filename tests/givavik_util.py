@@ -59,10 +59,10 @@ TINY = config([layer(latent(heads=2, dim=8, rot_dim=4, vdim=8, kv_rank=12), ff=1
                layer(parallel(left(heads=2, kv_heads=1, dim=8, vdim=12, dims=4), right(heads=2, vdim=8, state=8, groups=1, conv=3, norm_groups=1)), ff=None),
                layer(latent(heads=3, dim=12, rot_dim=4, vdim=4, kv_rank=12, kv_from=0), ff=24)], width=32, vocab=61, bigram=(17, 5, 3))
 #: values that a model may happen to make equal or one: one head, one group, one tap, factors and scale of one, no cap,
-#: no second table
+#: no second table; a width and a vocabulary that fit no vector access
 PLAIN = config([layer(parallel(left(heads=1, kv_heads=1, dim=16, vdim=16, scale=1.0, softcap=None, dims=16),
                                right(heads=1, vdim=16, state=16, groups=1, conv=1, norm_groups=1), 1.0, 1.0), ff=64),
-                layer(latent(heads=1, dim=16, rot_dim=16, vdim=16, kv_rank=16), ff=64)], width=64, vocab=90, scale=1.0, bigram=None)
+                layer(latent(heads=1, dim=16, rot_dim=16, vdim=16, kv_rank=16), ff=50)], width=66, vocab=91, scale=1.0, bigram=None)
 #: the head sizes of the serving kernels (keys and values of 64 and of 128, latent rows of 80 and 160: tensor cores for
 #: bfloat16); no two sizes alike where the kernels allow it
 SERVING_HEADS = config([layer(parallel(left(heads=6, kv_heads=2, dim=64, vdim=64, scale=0.12, softcap=30.0, dims=48, base=1e4),
