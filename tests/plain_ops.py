@@ -64,10 +64,12 @@ def add_residual(x, delta):
     x += _f(delta)
 
 
-def swiglu(g):
-    """crates/vapi-backend-candle/src/fused.rs:157-165."""
+def swiglu(g, act="silu"):
+    """crates/vapi-backend-candle/src/fused.rs:157-165; act "gelu_tanh": the tanh form of GELU on the gate."""
     f = g.shape[1] // 2
     a, b = _f(g[:, :f]), _f(g[:, f:])
+    if act == "gelu_tanh":
+        return (0.5 * a * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (a + 0.044715 * a ** 3))) * b).to(g.dtype)
     return ((a / (1.0 + torch.exp(-a))) * b).to(g.dtype)
 
 
@@ -734,8 +736,11 @@ def relu_squared(x):
     return (torch.relu(_f(x)) ** 2).to(x.dtype)
 
 
-def moe_route(h, router, correction, experts, top, groups, keep, bias=None, score="softmax"):
+def moe_route(h, router, correction, experts, top, groups, keep, bias=None, score="softmax", group_top=1, shared_gate=None):
     n = h.shape[0]
+    if shared_gate is not None:                       # the shared expert's gate: a last row of the router
+        shared_gate.copy_(torch.sigmoid(_f(h) @ router[-1]))
+        router = router[:-1]
     if score == "chosen":
         ids = torch.zeros((n, top), dtype=torch.int32)
         wts = torch.zeros((n, top), dtype=torch.float32)
@@ -750,10 +755,11 @@ def moe_route(h, router, correction, experts, top, groups, keep, bias=None, scor
     wts = torch.zeros((n, top), dtype=torch.float32)
     per = outputs // groups
     for t in range(n):
-        s = torch.softmax(router @ _f(h[t]) + (bias if bias is not None else 0.0), 0)
+        z = router @ _f(h[t]) + (bias if bias is not None else 0.0)
+        s = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, 0)
         choice = s + (correction if correction is not None else 0.0)
         if groups > 1 and keep < groups:
-            gs = choice.reshape(groups, per).max(1).values
+            gs = torch.sort(choice.reshape(groups, per), 1, descending=True).values[:, :group_top].sum(1)
             kept = sorted(range(groups), key=lambda g: (-float(gs[g]), g))[:keep]
             for g in range(groups):
                 if g not in kept:
@@ -770,7 +776,7 @@ def moe_table_route(tokens, table, experts, status=None):
     return ids, torch.full(ids.shape, 1.0 / ids.shape[1], dtype=torch.float32), None
 
 
-def moe_experts(h, ids, wts, plan, w_up, w_down, shared=None, gated=False, act=(0.0, 1.0, 0.0)):
+def moe_experts(h, ids, wts, plan, w_up, w_down, shared=None, gated=False, act=(0.0, 1.0, 0.0), shared_gate=None):
     """act = (limit, alpha, shift): a gated expert's hidden row is g' * sigmoid(alpha g') * (u' + shift) with g' = min(g, limit)
     and u' = clamp(u, -limit, limit) when limit > 0."""
     limit, alpha, shift = act
@@ -792,7 +798,7 @@ def moe_experts(h, ids, wts, plan, w_up, w_down, shared=None, gated=False, act=(
                 hid = (torch.relu(_f(w_up[e]) @ _f(h[t])) ** 2).to(h.dtype)
                 out[t] += g * (_f(w_down[e]) @ _f(hid))
     if shared is not None:
-        out += _f(shared)
+        out += _f(shared) * (shared_gate[:, None] if shared_gate is not None else 1.0)
     return out.to(h.dtype)
 
 
@@ -863,7 +869,31 @@ def gated_linear_attention(qkv, decay_logits, tau, state, state_slots, cu_q, pos
     return out
 
 
-ALL = ["matrix_memory", "gated_linear_attention", "embed", "resolve_tokens", "sample_truncated", "add_rmsnorm", "add_residual", "add_residual_ss", "skinny_applies", "tc_applies", "few_rows_applies", "swiglu", "linear", "strict_fp32", "rope_cos_sin",
+def fixed_decay_memory(qkv, powers, state, state_slots, cu_q, positions, nh, dk, dv, q_scale=1.0, act=None, status=None, max_q=1):
+    n = qkv.shape[0]
+    out = torch.zeros((n, nh * dv), dtype=torch.float32)
+    nS = nh * dk * dv
+    for s in range(cu_q.numel() - 1):
+        r0, r1 = int(cu_q[s]), int(cu_q[s + 1])
+        if r1 == r0:
+            continue
+        slot = int(state_slots[s])
+        S = state[slot, :nS].view(nh, dv, dk).transpose(1, 2).clone()          # the slot holds S column by column
+        if int(positions[r0]) == 0:
+            S.zero_()
+        for r in range(r0, r1):
+            row = _f(qkv[r])
+            if act == "silu":
+                row = row * torch.sigmoid(row)
+            q, k = row[:nh * dk].view(nh, dk), row[nh * dk:2 * nh * dk].view(nh, dk)
+            v = row[2 * nh * dk:2 * nh * dk + nh * dv].view(nh, dv)
+            S = powers[:, 1][:, None, None] * S + k[:, :, None] * v[:, None, :]
+            out[r] = q_scale * (S * q[:, :, None]).sum(1).reshape(-1)
+        state[slot, :nS] = S.transpose(1, 2).reshape(-1)
+    return out
+
+
+ALL = ["fixed_decay_memory", "matrix_memory", "gated_linear_attention", "embed", "resolve_tokens", "sample_truncated", "add_rmsnorm", "add_residual", "add_residual_ss", "skinny_applies", "tc_applies", "few_rows_applies", "swiglu", "linear", "strict_fp32", "rope_cos_sin",
        "qk_norm_rope_write", "attention_splits", "paged_attention", "shortconv", "sample_rows",
        "apply_penalties", "postnorm_add_rmsnorm", "gated_group_rmsnorm", "scale_rows", "rope_cos_sin_scaled",
        "qk_norm_rope_write_split", "masked_attention_splits", "masked_attention", "causal_conv_silu", "gated_delta",

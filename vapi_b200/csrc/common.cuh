@@ -171,6 +171,15 @@ __device__ __forceinline__ float xielu_16(float z, float up, float down) {
     return fmaf(0.5f, z, z > 0.f ? a * z : b);
 }
 
+// What the gate of a gated product passes: kind 0 is SiLU, z * sigmoid(z); kind 1 the tanh form of GELU,
+// 0.5 z (1 + tanh(u)) with u = sqrt(2/pi) (z + 0.044715 z^3), which is z * sigmoid(2u).
+__device__ __forceinline__ float glu_arg(float z, int kind) {
+    return kind ? z * fmaf(0.07135481627f * z, z, 1.595769122f) : z;
+}
+__device__ __forceinline__ float glu_gate(float z, int kind) { return z / (1.f + expf(-glu_arg(z, kind))); }
+// The same for results that are rounded to bfloat16 (fast exponential and division: their error is far below that rounding)
+__device__ __forceinline__ float glu_gate_16(float z, int kind) { return __fdividef(z, 1.f + __expf(-glu_arg(z, kind))); }
+
 // ---- warp / block reductions -----------------------------------------------
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

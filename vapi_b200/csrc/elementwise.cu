@@ -706,10 +706,10 @@ VAPI_EXPORT int vapi_add_residual(float* x, const void* delta, int dtype, long l
 
 // ---------------------------------------------------------------------------
 // SwiGLU on a stacked gate/up product: out[r, c] = silu(g[r, c]) * g[r, F + c],
-// silu(v) = v / (1 + exp(-v)); float math, one rounding
+// silu(v) = v / (1 + exp(-v)); float math, one rounding; `glu` names the gate's activation (glu_gate in common.cuh)
 // (crates/vapi-backend-candle/src/fused.rs:16-25, 157-165).
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ g, T* __restrict__ out, int rows, int ff) {
+__global__ void swiglu_kernel(const T* __restrict__ g, T* __restrict__ out, int rows, int ff, int glu) {
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     const size_t total = (size_t)rows * ff;
     const size_t stride = (size_t)gridDim.x * blockDim.x;
@@ -719,14 +719,13 @@ __global__ void swiglu_kernel(const T* __restrict__ g, T* __restrict__ out, int 
         const size_t r = i / ff, c = i - r * ff;
         const float a = to_f32(g[r * 2 * ff + c]);
         const float b = to_f32(g[r * 2 * ff + ff + c]);
-        const float s = a / (1.f + expf(-a));
-        out[i] = from_f32<T>(s * b);
+        out[i] = from_f32<T>(glu_gate(a, glu) * b);
     }
 }
 
 // four outputs per thread with 16-byte (float) / 8-byte (bfloat16) accesses; ff a multiple of 4
 template <typename T>
-__global__ void swiglu_vec_kernel(const T* __restrict__ g, T* __restrict__ out, int rows, int ff) {
+__global__ void swiglu_vec_kernel(const T* __restrict__ g, T* __restrict__ out, int rows, int ff, int glu) {
     const int f4 = ff >> 2;
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     const size_t total = (size_t)rows * f4;
@@ -737,14 +736,14 @@ __global__ void swiglu_vec_kernel(const T* __restrict__ g, T* __restrict__ out, 
         const size_t r = i / f4, c = (i - r * f4) << 2;
         const float4 a = Pack4<T>::load(g + r * 2 * ff + c);
         const float4 b = Pack4<T>::load(g + r * 2 * ff + ff + c);
-        Pack4<T>::store(out + r * ff + c, make_float4(a.x / (1.f + expf(-a.x)) * b.x, a.y / (1.f + expf(-a.y)) * b.y,
-                                                      a.z / (1.f + expf(-a.z)) * b.z, a.w / (1.f + expf(-a.w)) * b.w));
+        Pack4<T>::store(out + r * ff + c, make_float4(glu_gate(a.x, glu) * b.x, glu_gate(a.y, glu) * b.y,
+                                                      glu_gate(a.z, glu) * b.z, glu_gate(a.w, glu) * b.w));
     }
 }
 
 // bfloat16, ff a multiple of 8: one thread per eight outputs of one row, 16-byte accesses, no
 // loop and no index division (the row is the block's y index)
-__global__ void swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ g, __nv_bfloat16* __restrict__ out, int ff) {
+__global__ void swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ g, __nv_bfloat16* __restrict__ out, int ff, int glu) {
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) << 3;
     const size_t r = blockIdx.y;
     pdl_trigger();
@@ -758,14 +757,14 @@ __global__ void swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ g, __nv_b
     for (int i = 0; i < 4; ++i) {
         const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&aw[i]));
         const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&bw[i]));
-        __nv_bfloat162 y = __floats2bfloat162_rn(x.x / (1.f + expf(-x.x)) * u.x, x.y / (1.f + expf(-x.y)) * u.y);
+        __nv_bfloat162 y = __floats2bfloat162_rn(glu_gate(x.x, glu) * u.x, glu_gate(x.y, glu) * u.y);
         o[i] = *reinterpret_cast<unsigned*>(&y);
     }
     *reinterpret_cast<uint4*>(out + r * ff + c) = make_uint4(o[0], o[1], o[2], o[3]);
 }
 
 VAPI_EXPORT int vapi_swiglu(const void* g, void* out, int dtype, int rows, int ff,
-                            cudaStream_t stream) {
+                            cudaStream_t stream, int glu) {
     if (rows <= 0) return 0;
     if (ff <= 0) return fail(-1, "swiglu: ff=%d", ff);
     const int threads = 256;
@@ -776,20 +775,20 @@ VAPI_EXPORT int vapi_swiglu(const void* g, void* out, int dtype, int rows, int f
     if (dtype == VAPI_BF16 && ff % 8 == 0 && rows <= 65535) {
         const int th = 128;
         dim3 grid((ff / 8 + th - 1) / th, rows);
-        e = launch(swiglu_bf16x8_kernel, grid, th, 0, stream, (const __nv_bfloat16*)g, (__nv_bfloat16*)out, ff);
+        e = launch(swiglu_bf16x8_kernel, grid, th, 0, stream, (const __nv_bfloat16*)g, (__nv_bfloat16*)out, ff, glu);
         return check_launch("swiglu", e);
     }
     if (ff % 4 == 0 && (dtype == VAPI_F32 || dtype == VAPI_BF16)) {
         long long vb = (total / 4 + threads - 1) / threads;
         if (vb > sm_count() * 16) vb = sm_count() * 16;
-        if (dtype == VAPI_F32) e = launch(swiglu_vec_kernel<float>, (int)vb, threads, 0, stream, (const float*)g, (float*)out, rows, ff);
-        else e = launch(swiglu_vec_kernel<__nv_bfloat16>, (int)vb, threads, 0, stream, (const __nv_bfloat16*)g, (__nv_bfloat16*)out, rows, ff);
+        if (dtype == VAPI_F32) e = launch(swiglu_vec_kernel<float>, (int)vb, threads, 0, stream, (const float*)g, (float*)out, rows, ff, glu);
+        else e = launch(swiglu_vec_kernel<__nv_bfloat16>, (int)vb, threads, 0, stream, (const __nv_bfloat16*)g, (__nv_bfloat16*)out, rows, ff, glu);
         return check_launch("swiglu", e);
     }
     if (dtype == VAPI_F32)
-        e = launch(swiglu_kernel<float>, (int)blocks, threads, 0, stream, (const float*)g, (float*)out, rows, ff);
+        e = launch(swiglu_kernel<float>, (int)blocks, threads, 0, stream, (const float*)g, (float*)out, rows, ff, glu);
     else if (dtype == VAPI_BF16)
-        e = launch(swiglu_kernel<__nv_bfloat16>, (int)blocks, threads, 0, stream, (const __nv_bfloat16*)g, (__nv_bfloat16*)out, rows, ff);
+        e = launch(swiglu_kernel<__nv_bfloat16>, (int)blocks, threads, 0, stream, (const __nv_bfloat16*)g, (__nv_bfloat16*)out, rows, ff, glu);
     else
         return fail(-2, "swiglu: unsupported dtype %d", dtype);
     return check_launch("swiglu", e);

@@ -81,6 +81,7 @@ struct GvParams {
     __nv_bfloat16* out_bf16; float* out_f32; long long out_stride;
     const float* bias;
     const float* xielu;                            // EPI_BF16: null, or {up, down}: the output passes xIELU
+    int glu;                                       // EPI_SWIGLU: the gate's activation (glu_gate)
     float* resid; float* ss_out;                   // EPI_RESID
     const float* next_w; __nv_bfloat16* xw_out;    // EPI_RESID: weight of the norm that follows, [M][N] out
     int ff;                                        // EPI_SWIGLU: N == 2*ff
@@ -255,7 +256,7 @@ __device__ __forceinline__ void gv_tile_finish(const GvParams& p, int tile, int 
     } else if (EPI == GV_EPI_SWIGLU) {
         const long long col = (long long)tile * 8 + i;
         if (i < 8 && m < p.M && col < p.ff) {
-            const float sg = y / (1.f + expf(-y));
+            const float sg = glu_gate(y, p.glu);
             p.out_bf16[(size_t)m * p.out_stride + col] = __float2bfloat16_rn(sg * y2);
         }
     } else {
@@ -786,7 +787,7 @@ VAPI_EXPORT int vapi_skinny_linear(const void* W, int N, int K, int M, int pro, 
                                    int epi, void* out_bf16, float* out_f32, long long out_stride,
                                    const float* bias, float* resid, float* ss_out,
                                    const float* next_w, void* xw_out, int rows_per_cta,
-                                   cudaStream_t stream, const float* xielu_consts) {
+                                   cudaStream_t stream, const float* xielu_consts, int glu) {
     if (M <= 0) return 0;
     if (xielu_consts && epi != GV_EPI_BF16) return fail(-1, "skinny_linear: xIELU comes with the bfloat16 output");
     if (M > 16) return fail(-1, "skinny_linear: %d rows are more than 16", M);
@@ -804,7 +805,7 @@ VAPI_EXPORT int vapi_skinny_linear(const void* W, int N, int K, int M, int pro, 
     p.act = (const __nv_bfloat16*)act; p.xw = (const __nv_bfloat16*)xw; p.ss_in = ss_in; p.ss_parts = ss_parts; p.eps = eps;
     p.next_w = next_w; p.xw_out = (__nv_bfloat16*)xw_out;
     p.out_bf16 = (__nv_bfloat16*)out_bf16; p.out_f32 = out_f32; p.out_stride = out_stride; p.bias = bias;
-    p.xielu = xielu_consts;
+    p.xielu = xielu_consts; p.glu = glu;
     p.resid = resid; p.ss_out = ss_out; p.ff = N / 2; p.rows_per_cta = epi == GV_EPI_SWIGLU ? 16 : rows_per_cta;
     const int blocks = vapi_skinny_linear_blocks(N, epi, rows_per_cta);
     p.num_tiles = blocks;

@@ -61,6 +61,7 @@ struct PlParams {
     const float* bias; float* resid; float* ss_out; const float* next_w; __nv_bfloat16* xw_out;
     int* status;
     const float* xielu;                            // EPI_BF16: null, or {up, down}: the output passes xIELU
+    int glu;                                       // EPI_SWIGLU: the gate's activation (glu_gate)
 };
 
 template <int BN, int PAIR> struct PlCfg {
@@ -326,8 +327,7 @@ prompt_linear_kernel(const __grid_constant__ CUtensorMap tm_a, const __grid_cons
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
                         const float gv = __uint_as_float(g[j]) * scale, uv = __uint_as_float(u[j]) * scale;
-                        // (fast exponential and division: their error is far below the bfloat16 rounding of the result)
-                        sv[j] = __fdividef(gv, 1.f + __expf(-gv)) * uv;
+                        sv[j] = glu_gate_16(gv, p.glu) * uv;
                     }
                     if (vec_out && f0 + 31 < p.ff) {
                         put(sv);
@@ -571,7 +571,7 @@ VAPI_EXPORT int vapi_prompt_linear(const void* W, int N, int K, int M, int pro, 
                                    const float* ss_in, int ss_parts, float eps, int epi, void* out_bf16,
                                    float* out_f32, long long out_stride, const float* bias, float* resid,
                                    float* ss_out, const float* next_w, void* xw_out, int* status,
-                                   cudaStream_t stream, const float* xielu_consts) {
+                                   cudaStream_t stream, const float* xielu_consts, int glu) {
     if (M <= 0) return 0;
     if (xielu_consts && epi != PL_EPI_BF16) return fail(-1, "prompt_linear: xIELU comes with the bfloat16 output");
     if (N <= 0 || K <= 0 || K % 8 != 0) return fail(-1, "prompt_linear: K=%d must be a positive multiple of 8 (N=%d)", K, N);
@@ -595,7 +595,7 @@ VAPI_EXPORT int vapi_prompt_linear(const void* W, int N, int K, int M, int pro, 
     p.ss_in = ss_in; p.ss_parts = ss_parts; p.eps = eps;
     p.out_bf16 = (__nv_bfloat16*)out_bf16; p.out_f32 = out_f32; p.out_stride = out_stride; p.bias = bias;
     p.resid = resid; p.ss_out = ss_out; p.next_w = next_w; p.xw_out = (__nv_bfloat16*)xw_out;
-    p.status = status; p.xielu = xielu_consts;
+    p.status = status; p.xielu = xielu_consts; p.glu = glu;
     const bool half_rows = epi == PL_EPI_SWIGLU || pair == 2;      // boxes of BN/2 weight rows
     const CUtensorMap *ta, *tw;
     int rc = pl_map(&ta, tokens, M, K, PL_BM);

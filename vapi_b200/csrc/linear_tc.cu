@@ -46,6 +46,7 @@ struct TcParams {
     const float* bias; float* resid; float* ss_out; const float* next_w; __nv_bfloat16* xw_out;
     int* status;
     const float* xielu;                                            // EPI_BF16: null, or {up, down}: the output passes xIELU
+    int glu;                                                       // EPI_SWIGLU: the gate's activation (glu_gate)
 };
 
 template <int BN> struct TcCfg {
@@ -187,8 +188,7 @@ linear_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant
             // 64 features: gate in rows 0..63, up in rows 64..127; two features per lane
             const long long f0 = (long long)n0 + 2 * lane;
             const float g0 = f[2 * lane], g1 = f[2 * lane + 1], u0 = f[64 + 2 * lane], u1 = f[64 + 2 * lane + 1];
-            // (fast exponential and division: their error is far below the bfloat16 rounding of the result)
-            const float s0 = __fdividef(g0, 1.f + __expf(-g0)) * u0, s1 = __fdividef(g1, 1.f + __expf(-g1)) * u1;
+            const float s0 = glu_gate_16(g0, p.glu) * u0, s1 = glu_gate_16(g1, p.glu) * u1;
             __nv_bfloat16* o = p.out_bf16 + (size_t)m * p.out_stride + f0;
             if (f0 + 1 < p.ff && (p.out_stride & 1) == 0) *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(s0, s1);
             else {
@@ -405,7 +405,7 @@ VAPI_EXPORT int vapi_linear_tc(const void* W, int N, int K, int M, int pro, cons
                                const float* ss_in, int ss_parts, float eps, int epi, void* out_bf16,
                                float* out_f32, long long out_stride, const float* bias, float* resid,
                                float* ss_out, const float* next_w, void* xw_out, int* status,
-                               cudaStream_t stream, const float* xielu_consts) {
+                               cudaStream_t stream, const float* xielu_consts, int glu) {
     if (M <= 0) return 0;
     if (xielu_consts && epi != TC_EPI_BF16) return fail(-1, "linear_tc: xIELU comes with the bfloat16 output");
     if (M > 256) return fail(-1, "linear_tc: %d rows are more than 256", M);
@@ -425,7 +425,7 @@ VAPI_EXPORT int vapi_linear_tc(const void* W, int N, int K, int M, int pro, cons
     p.ss_in = ss_in; p.ss_parts = ss_parts; p.eps = eps;
     p.out_bf16 = (__nv_bfloat16*)out_bf16; p.out_f32 = out_f32; p.out_stride = out_stride; p.bias = bias;
     p.resid = resid; p.ss_out = ss_out; p.next_w = next_w; p.xw_out = (__nv_bfloat16*)xw_out;
-    p.status = status; p.xielu = xielu_consts;
+    p.status = status; p.xielu = xielu_consts; p.glu = glu;
     CUtensorMap tw, ta;
     int rc = make_map(&tw, W, N, K, epi == TC_EPI_SWIGLU ? 64 : TC_BM);
     if (rc) return rc;

@@ -8,7 +8,10 @@
 // lower index); their weights are their s divided by the sum of the chosen s (+ 1e-20).  An output
 // index >= experts is an identity expert: its output is the input itself.
 // A second way of scoring (score_mode 1): the choice is made among the logits z = Wr h + bias themselves, and the
-// weights are the softmax over the chosen logits only.
+// weights are the softmax over the chosen logits only.  A third (score_mode 2): s = sigmoid(z), output by output.  With
+// group_top 2 a group's score is the sum of its two largest choice scores (of its only one, where it has no second).
+// A shared expert's gate may ride along: one more row behind the router's, whose product goes through a sigmoid to
+// shared_gate[t], by which the sum below multiplies the shared expert's output.
 //
 // The step's expert work is laid out without the host learning anything about it: after the router, one
 // block counts the (token, choice) pairs of each expert in shared memory (a pair's rank within its expert is
@@ -50,24 +53,25 @@ template <> struct RtLd4<__nv_bfloat16> {
 // One block of four warps per token: the warps share the router's outputs among them (four outputs at a time
 // a warp, so that a lane has their loads in flight together), then the first warp chooses.  The order of a
 // lane's additions and of a warp's reduction depends on nothing but the width.  shared memory: 2 * outputs
-// floats (the scores and the choice scores) + groups floats.
+// floats (the scores and the choice scores) + groups floats + one (the shared expert's gate).
 template <typename T>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ corr,
                  const float* __restrict__ bias, int score_mode,
                  int* __restrict__ ids, float* __restrict__ wts, int n, int width, int outputs, int experts, int top,
-                 int groups, int keep, int vec4) {
+                 int groups, int keep, int vec4, int group_top, float* __restrict__ shared_gate) {
     extern __shared__ float rt_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int t = blockIdx.x;
     float* s = rt_smem;
-    float* choice = s + outputs;
+    const int nrows = outputs + (shared_gate ? 1 : 0);         // the router's rows, and the shared expert's gate
+    float* choice = s + outputs + 1;
     float* gscore = choice + outputs;
     pdl_trigger();
     pdl_wait();
     if (t >= n) return;
     const T* hr = h + (size_t)t * width;
-    for (int e0 = warp * 4; e0 < outputs; e0 += warps * 4) {
+    for (int e0 = warp * 4; e0 < nrows; e0 += warps * 4) {
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
         const float* w0 = wr + (size_t)e0 * width;
         if (vec4) {
@@ -75,7 +79,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const fl
                 const float4 hv = RtLd4<T>::load(hr + k);
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
-                    if (e0 + j < outputs) {
+                    if (e0 + j < nrows) {
                         const float4 wv = *reinterpret_cast<const float4*>(w0 + (size_t)j * width + k);
                         acc[j] = fmaf(hv.x, wv.x, acc[j]);
                         acc[j] = fmaf(hv.y, wv.y, acc[j]);
@@ -89,13 +93,13 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const fl
                 const float hv = to_f32(hr[k]);
 #pragma unroll
                 for (int j = 0; j < 4; ++j)
-                    if (e0 + j < outputs) acc[j] = fmaf(hv, w0[(size_t)j * width + k], acc[j]);
+                    if (e0 + j < nrows) acc[j] = fmaf(hv, w0[(size_t)j * width + k], acc[j]);
             }
         }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const float v = warp_sum(acc[j]);
-            if (lane == 0 && e0 + j < outputs) s[e0 + j] = bias ? v + bias[e0 + j] : v;
+            if (lane == 0 && e0 + j < nrows) s[e0 + j] = bias && e0 + j < outputs ? v + bias[e0 + j] : v;
         }
     }
     __syncthreads();
@@ -103,8 +107,15 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const fl
     {
 
     __syncwarp();
+    if (shared_gate && lane == 0) shared_gate[t] = 1.f / (1.f + expf(-s[outputs]));
     if (score_mode == 1) {
         for (int e = lane; e < outputs; e += 32) choice[e] = s[e];
+    } else if (score_mode == 2) {
+        for (int e = lane; e < outputs; e += 32) {
+            const float p = 1.f / (1.f + expf(-s[e]));
+            s[e] = p;
+            choice[e] = p + (corr ? corr[e] : 0.f);
+        }
     } else {
     float mx = -INFINITY;
     for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, s[e]);
@@ -122,9 +133,12 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const fl
     if (groups > 1 && keep < groups) {
         const int per = outputs / groups;
         for (int gi = lane; gi < groups; gi += 32) {
-            float m = -INFINITY;
-            for (int e = gi * per; e < (gi + 1) * per; ++e) m = fmaxf(m, choice[e]);
-            gscore[gi] = m;
+            float m = -INFINITY, second = -INFINITY;
+            for (int e = gi * per; e < (gi + 1) * per; ++e) {
+                second = fmaxf(second, fminf(m, choice[e]));
+                m = fmaxf(m, choice[e]);
+            }
+            gscore[gi] = group_top == 2 && per > 1 ? m + second : m;
         }
         __syncwarp();
         // the best `keep` groups, one after the other; a chosen group is marked by +inf
@@ -433,22 +447,23 @@ moe_grouped_mma_kernel(const __nv_bfloat16* __restrict__ A, long long a_stride, 
 }
 
 // out[t, :] = sum over the token's choices (an expert's row of y, or weight * h for an identity expert)
-// + shared[t, :] (when given), in the order of the choices.
+// + shared[t, :] (when given, times shared_gate[t]), in the order of the choices.
 template <typename T>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ ids, const float* __restrict__ wts,
                                    const T* __restrict__ h, const T* __restrict__ shared, T* __restrict__ out, int n,
-                                   int width, int top, int experts) {
+                                   int width, int top, int experts, const float* __restrict__ shared_gate) {
     const int t = blockIdx.x;
     pdl_trigger();
     pdl_wait();
     if (t >= n) return;
+    const float gate = shared_gate ? shared_gate[t] : 1.f;
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         float acc = 0.f;
         for (int r = 0; r < top; ++r) {
             const size_t p = (size_t)t * top + r;
             acc += ids[p] < experts ? y[p * width + c] : wts[p] * to_f32(h[(size_t)t * width + c]);
         }
-        if (shared) acc += to_f32(shared[(size_t)t * width + c]);
+        if (shared) acc = fmaf(gate, to_f32(shared[(size_t)t * width + c]), acc);
         out[(size_t)t * width + c] = from_f32<T>(acc);
     }
 }
@@ -500,23 +515,26 @@ VAPI_EXPORT int vapi_relu_squared(const void* x, void* out, int dtype, long long
 VAPI_EXPORT int vapi_moe_route(const void* h, int dtype, const float* wr, const float* corr, const float* bias,
                                int score_mode, int* ids, float* wts, int* ranks,
                                int* offsets, int* pair_of, int* plan, int* tile_expert, int* tile_row0, int n,
-                               int width, int outputs, int experts, int top, int groups, int keep, cudaStream_t stream) {
+                               int width, int outputs, int experts, int top, int groups, int keep, cudaStream_t stream,
+                               int group_top, float* shared_gate) {
     if (n <= 0) return 0;
+    if (score_mode < 0 || score_mode > 2 || group_top < 1 || group_top > 2)
+        return fail(-1, "moe_route: score mode %d, a group's score from its %d largest", score_mode, group_top);
     if (outputs <= 0 || experts < 0 || experts > outputs || top <= 0 || top > outputs)
         return fail(-1, "moe_route: %d outputs, %d experts, top %d", outputs, experts, top);
     if (groups < 1 || outputs % groups || keep < 1 || keep > groups)
         return fail(-1, "moe_route: %d outputs in %d groups, %d kept", outputs, groups, keep);
     if ((long long)(outputs / groups) * keep < top) return fail(-1, "moe_route: %d kept groups cannot give %d choices", keep, top);
     cudaError_t e;
-    const size_t smem = (size_t)(2 * outputs + groups) * sizeof(float);
+    const size_t smem = (size_t)(2 * outputs + groups + 1) * sizeof(float);
     if (smem > 48 * 1024) return fail(-1, "moe_route: %d router outputs are too many", outputs);
     const int vec4 = (width % 4 == 0 && ((uintptr_t)h & 15) == 0 && ((uintptr_t)wr & 15) == 0) ? 1 : 0;
     if (dtype == VAPI_F32)
         e = launch(moe_route_kernel<float>, n, 128, smem, stream, (const float*)h, wr, corr, bias, score_mode, ids, wts, n,
-                   width, outputs, experts, top, groups, keep, vec4);
+                   width, outputs, experts, top, groups, keep, vec4, group_top, shared_gate);
     else if (dtype == VAPI_BF16)
         e = launch(moe_route_kernel<__nv_bfloat16>, n, 128, smem, stream, (const __nv_bfloat16*)h, wr, corr, bias, score_mode, ids,
-                   wts, n, width, outputs, experts, top, groups, keep, vec4);
+                   wts, n, width, outputs, experts, top, groups, keep, vec4, group_top, shared_gate);
     else
         return fail(-2, "moe_route: unsupported dtype %d", dtype);
     int rc = check_launch("moe_route", e);
@@ -593,16 +611,17 @@ VAPI_EXPORT int vapi_moe_grouped(const void* A, long long a_stride, const void* 
 }
 
 VAPI_EXPORT int vapi_moe_combine(const float* y, const int* ids, const float* wts, const void* h, const void* shared,
-                                 void* out, int dtype, int n, int width, int top, int experts, cudaStream_t stream) {
+                                 void* out, int dtype, int n, int width, int top, int experts, cudaStream_t stream,
+                                 const float* shared_gate) {
     if (n <= 0) return 0;
     const int threads = width >= 1024 ? 256 : 128;
     cudaError_t e;
     if (dtype == VAPI_F32)
         e = launch(moe_combine_kernel<float>, n, threads, 0, stream, y, ids, wts, (const float*)h, (const float*)shared,
-                   (float*)out, n, width, top, experts);
+                   (float*)out, n, width, top, experts, shared_gate);
     else if (dtype == VAPI_BF16)
         e = launch(moe_combine_kernel<__nv_bfloat16>, n, threads, 0, stream, y, ids, wts, (const __nv_bfloat16*)h,
-                   (const __nv_bfloat16*)shared, (__nv_bfloat16*)out, n, width, top, experts);
+                   (const __nv_bfloat16*)shared, (__nv_bfloat16*)out, n, width, top, experts, shared_gate);
     else
         return fail(-2, "moe_combine: unsupported dtype %d", dtype);
     return check_launch("moe_combine", e);

@@ -30,12 +30,12 @@ e<j>.down, table}``, ``final.norm``.
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Any, Dict, List, Optional, Tuple
+from typing import Any, Dict, Optional, Tuple
 
 from ..config.model import Architecture, ConfigError, register_architecture, require_int
 from ..parts import (GQAttention, LatentAttention, OutputHead, ParallelBlock, RGLRUMixer, RMSNorm, ScaledRotaryEncoding,
                      SparseMoE, StreamInjection, TokenEmbedding)
-from .plan import LayerCall, ModelPlan
+from .plan import ModelPlan, looped_order
 
 #: positions are counted in float32, which holds integers exactly up to here
 MAX_POSITIONS = 1 << 24
@@ -146,17 +146,6 @@ class NelosunConfig:
                    embedding_scale=scale, loop=loop, layers=tuple(layers), eos_token_ids=tuple(sorted(set(eos_ids))))
 
 
-def run_order(n_layers: int, loop: Optional[Tuple[int, int, int]], inject: str) -> List[LayerCall]:
-    """Every layer once, but those of the loop ``times`` times in a row, each pass led by the stream part."""
-    if loop is None:
-        return [LayerCall(i) for i in range(n_layers)]
-    a, b, times = loop
-    order = [LayerCall(i) for i in range(a)]
-    for _ in range(times):
-        order += [LayerCall(i, before=inject if i == a else None) for i in range(a, b)]
-    return order + [LayerCall(i) for i in range(b, n_layers)]
-
-
 def nelosun_plan(cfg: NelosunConfig) -> ModelPlan:
     W, eps = cfg.width, cfg.norm_eps
     emb = TokenEmbedding(cfg.vocab, W, "embed", scale=cfg.embedding_scale)
@@ -192,7 +181,7 @@ def nelosun_plan(cfg: NelosunConfig) -> ModelPlan:
     stream_parts = {"loop_in": StreamInjection(W, "loop.in")} if cfg.loop is not None else {}
     return ModelPlan(
         architecture="Nelosun", vocab_size=cfg.vocab, hidden_size=W, max_positions=MAX_POSITIONS, embedding=emb,
-        layers=layers, layer_prefixes=prefixes, order=run_order(len(layers), cfg.loop, "loop_in"),
+        layers=layers, layer_prefixes=prefixes, order=looped_order(len(layers), cfg.loop, "loop_in"),
         final_norm=RMSNorm(W, eps, "norm"), final_norm_prefix="final.",
         head=OutputHead(cfg.vocab, W, True, emb, "head"),
         position_encodings=list(ropes.values()), eos_token_ids=cfg.eos_token_ids, config=cfg, stream_parts=stream_parts)

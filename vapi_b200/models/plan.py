@@ -26,6 +26,18 @@ class LayerCall:
     before: Optional[str] = None
 
 
+def looped_order(n_layers: int, loop: Optional[Tuple[int, int, int]], before: Optional[str] = None) -> List[LayerCall]:
+    """Every layer once, but those of ``loop`` = (start, stop, times) that many times in a row (each pass with caches of its
+    own), each pass led by the stream part ``before`` names."""
+    if loop is None:
+        return [LayerCall(i) for i in range(n_layers)]
+    a, b, times = loop
+    order = [LayerCall(i) for i in range(a)]
+    for _ in range(times):
+        order += [LayerCall(i, before=before if i == a else None) for i in range(a, b)]
+    return order + [LayerCall(i) for i in range(b, n_layers)]
+
+
 @dataclass
 class ModelPlan:
     architecture: str

@@ -291,8 +291,18 @@ def add_residual(x: torch.Tensor, delta: torch.Tensor) -> None:
     _check(lib, lib.vapi_add_residual(_p(x), _p(delta), _dt(delta), ctypes.c_longlong(x.numel()), _stream()))
 
 
-def swiglu(g: torch.Tensor) -> torch.Tensor:
-    """``silu(g[:, :F]) * g[:, F:]`` for a stacked gate/up product [n, 2F]."""
+#: what a gate passes in the gated products (see csrc/common.cuh)
+_GLU = {"silu": 0, "gelu_tanh": 1}
+
+
+def _glu(act: str) -> int:
+    if act not in _GLU:
+        raise KernelError(f"activation `{act}` is not one of {', '.join(_GLU)}")
+    return _GLU[act]
+
+
+def swiglu(g: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """``act(g[:, :F]) * g[:, F:]`` for a stacked gate/up product [n, 2F]; ``act`` is "silu" or "gelu_tanh" (the tanh form)."""
     _cuda(g)
     _contig(g, "gate/up product")
     rows, two_f = g.shape
@@ -300,7 +310,7 @@ def swiglu(g: torch.Tensor) -> torch.Tensor:
         raise KernelError("swiglu needs an even number of columns")
     out = torch.empty((rows, two_f // 2), dtype=g.dtype, device=g.device)
     lib = _lib("elementwise")
-    _check(lib, lib.vapi_swiglu(_p(g), _p(out), _dt(g), rows, two_f // 2, _stream()))
+    _check(lib, lib.vapi_swiglu(_p(g), _p(out), _dt(g), rows, two_f // 2, _stream(), _glu(act)))
     return out
 
 
@@ -336,14 +346,14 @@ def skinny_linear(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None,
                   xw: Optional[torch.Tensor] = None, ss_in: Optional[torch.Tensor] = None, eps: float = 0.0,
                   epilogue: str = "bf16", bias: Optional[torch.Tensor] = None,
                   resid: Optional[torch.Tensor] = None, next_weight: Optional[torch.Tensor] = None,
-                  rows_per_block: Optional[int] = None, xielu: Optional[torch.Tensor] = None):
+                  rows_per_block: Optional[int] = None, xielu: Optional[torch.Tensor] = None, glu: str = "silu"):
     """The weight-streaming product for decode steps (at most 16 rows), with its fusions.
 
     Token operand: ``act`` [M, K] bfloat16; or the residual stream seen through an RMSNorm not
     applied yet: ``xw`` [M, K] = bfloat16(stream * norm weight) with the partial sums of squares
     ``ss_in`` [parts, M] of the stream's rows (both left by whoever wrote the stream last) and the
     norm's ``eps``.  ``epilogue``: "bf16" -> [M, N] bfloat16; "f32" -> [M, N] float32; "swiglu" ->
-    [M, N/2] bfloat16 = silu(first half) * second half; "resid" -> adds into ``resid`` [M, N]
+    [M, N/2] bfloat16 = silu(first half) * second half (``glu`` "gelu_tanh": the tanh form of GELU instead); "resid" -> adds into ``resid`` [M, N]
     float32 in place and returns ``(ss, xw)`` of the new stream for the norm whose weight is
     ``next_weight`` (``(None, None)`` without it).  ``xielu`` [2] float32 (see :func:`xielu`), with the epilogue "bf16":
     the output passes the activation before it is rounded.
@@ -389,7 +399,7 @@ def skinny_linear(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None,
     _check(lib, lib.vapi_skinny_linear(
         _p(weight), N, K, M, _PRO[pro], _p(act), _p(xw), _p(ss_in), 0 if ss_in is None else ss_in.shape[0],
         ctypes.c_float(eps), _EPI[epilogue], _p(out_bf16), _p(out_f32), ctypes.c_longlong(out_stride), _p(bias),
-        _p(resid), _p(sso), _p(next_weight), _p(xwo), rpb, _stream(), _p(xielu)))
+        _p(resid), _p(sso), _p(next_weight), _p(xwo), rpb, _stream(), _p(xielu), _glu(glu)))
     if epilogue == "resid":
         return sso, xwo
     return out_bf16 if out_bf16 is not None else out_f32
@@ -469,7 +479,7 @@ def _tc_plan(N: int, K: int, M: int, epi: int):
 
 
 def _fused_product(which: str, weight: torch.Tensor, act, xw, ss_in, eps: float, epilogue: str, bias, resid,
-                   next_weight, status, xielu=None):
+                   next_weight, status, xielu=None, glu: str = "silu"):
     """Operand checks, outputs and the call shared by :func:`linear_tc` and :func:`prompt_linear`."""
     _cuda(weight, act, xw, ss_in, bias, resid, next_weight, xielu)
     _f32(xielu, "the activation's numbers")
@@ -517,7 +527,7 @@ def _fused_product(which: str, weight: torch.Tensor, act, xw, ss_in, eps: float,
     _check(lib, fn(
         _p(weight), N, K, M, _PRO[pro], _p(src), _p(ss_in), 0 if ss_in is None else ss_in.shape[0], ctypes.c_float(eps),
         _EPI[epilogue], _p(out_bf16), _p(out_f32), ctypes.c_longlong(out_stride), _p(bias), _p(resid), _p(sso),
-        _p(next_weight), _p(xwo), _p(status), _stream(), _p(xielu)))
+        _p(next_weight), _p(xwo), _p(status), _stream(), _p(xielu), _glu(glu)))
     if epilogue == "resid":
         return sso, xwo
     return out_bf16 if out_bf16 is not None else out_f32
@@ -527,10 +537,10 @@ def linear_tc(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None, xw: O
               ss_in: Optional[torch.Tensor] = None, eps: float = 0.0, epilogue: str = "bf16",
               bias: Optional[torch.Tensor] = None, resid: Optional[torch.Tensor] = None,
               next_weight: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None,
-              xielu: Optional[torch.Tensor] = None):
+              xielu: Optional[torch.Tensor] = None, glu: str = "silu"):
     """The tcgen05 / TMA product for 17..256 rows; same operands, epilogues and results as
     :func:`skinny_linear`."""
-    return _fused_product("linear_tc", weight, act, xw, ss_in, eps, epilogue, bias, resid, next_weight, status, xielu)
+    return _fused_product("linear_tc", weight, act, xw, ss_in, eps, epilogue, bias, resid, next_weight, status, xielu, glu)
 
 
 #: steps of more rows than TC_MAX_ROWS go to the persistent tcgen05 product of csrc/linear_prompt.cu
@@ -559,18 +569,18 @@ def _prompt_plan(N: int, K: int, M: int, epi: int):
 PROMPT_SWIGLU_MIN_ROWS = int(os.environ.get("VAPI_PROMPT_SWIGLU_MIN_ROWS", "256"))
 
 
-def linear_swiglu(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
-    """``silu(x @ Wg.T) * (x @ Wu.T)`` for ``weight = [Wg; Wu]``: one kernel with SwiGLU as the
+def linear_swiglu(x: torch.Tensor, weight: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """``act(x @ Wg.T) * (x @ Wu.T)`` for ``weight = [Wg; Wu]`` (``act`` "silu" or "gelu_tanh"): one kernel with the gate as the
     product's epilogue for prompt-sized bfloat16 steps, else the product followed by :func:`swiglu`."""
     rows = x.shape[0]
     if (x.dtype == torch.bfloat16 and 0 < PROMPT_SWIGLU_MIN_ROWS <= rows and rows > TC_MAX_ROWS and weight.is_cuda
             and weight.dtype == torch.bfloat16 and weight.dim() == 2 and weight.shape[1] % 8 == 0 and weight.shape[0] % 16 == 0
             and weight.is_contiguous() and x.is_contiguous()):
-        return prompt_linear(weight, act=x, epilogue="swiglu")
+        return prompt_linear(weight, act=x, epilogue="swiglu", glu=act)
     if (x.dtype == torch.bfloat16 and x.is_contiguous() and weight.shape[0] % 16 == 0 and rows <= TC_MAX_ROWS
             and few_rows_applies(rows, weight)):
-        return few_rows_linear(weight, act=x, epilogue="swiglu")      # a decode step: SwiGLU rides on the product
-    return swiglu(linear(x, weight))
+        return few_rows_linear(weight, act=x, epilogue="swiglu", glu=act)      # a decode step: the gate rides on the product
+    return swiglu(linear(x, weight), act)
 
 
 #: a product with xIELU behind it goes to the persistent tcgen05 product from this many rows on (0: never); below, the
@@ -614,10 +624,10 @@ def prompt_linear(weight: torch.Tensor, *, act: Optional[torch.Tensor] = None, x
                   ss_in: Optional[torch.Tensor] = None, eps: float = 0.0, epilogue: str = "bf16",
                   bias: Optional[torch.Tensor] = None, resid: Optional[torch.Tensor] = None,
                   next_weight: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None,
-                  xielu: Optional[torch.Tensor] = None):
+                  xielu: Optional[torch.Tensor] = None, glu: str = "silu"):
     """The persistent tcgen05 / TMA product for prompt-sized steps; same operands, epilogues and
     results as :func:`skinny_linear`."""
-    return _fused_product("linear_prompt", weight, act, xw, ss_in, eps, epilogue, bias, resid, next_weight, status, xielu)
+    return _fused_product("linear_prompt", weight, act, xw, ss_in, eps, epilogue, bias, resid, next_weight, status, xielu, glu)
 
 
 def few_rows_applies(rows: int, weight: torch.Tensor) -> bool:
@@ -1789,8 +1799,12 @@ def relu_squared(x: torch.Tensor) -> torch.Tensor:
     return out
 
 
+_SCORES = {"softmax": 0, "chosen": 1, "sigmoid": 2}
+
+
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], experts: int, top: int, groups: int,
-              keep: int, bias: Optional[torch.Tensor] = None, score: str = "softmax"):
+              keep: int, bias: Optional[torch.Tensor] = None, score: str = "softmax", group_top: int = 1,
+              shared_gate: Optional[torch.Tensor] = None):
     """The router of a mixture of experts for ``h`` [n, W]: ``router`` [outputs, W] and ``correction`` [outputs]
     float32, ``outputs`` = ``experts`` + identity experts.  Scores are the softmax of the float32 logits over all
     outputs; the ``top`` largest of score + correction win, among the outputs of the ``keep`` best of ``groups``
@@ -1798,17 +1812,22 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.
     scores divided by their sum (+ 1e-20).  Returns ``(ids [n, top] int32, weights [n, top] float32, plan)``;
     ``plan`` lists the step's (token, choice) pairs expert by expert for :func:`moe_experts`.  ``bias`` [outputs] is
     added to the logits.  ``score`` "chosen": the ``top`` largest logits win and the weights are the softmax over
-    the chosen logits only (no correction)."""
-    _cuda(h, router, correction, bias)
+    the chosen logits only (no correction); "sigmoid": scores are the logits' sigmoids.  ``group_top`` 2: a group's score is
+    the sum of its two largest.  ``shared_gate`` [n] float32, when given, receives ``sigmoid(w_g . h)`` with w_g a last
+    row of ``router`` behind the outputs' (the gate of a shared expert, see :func:`moe_experts`)."""
+    _cuda(h, router, correction, bias, shared_gate)
     _f32(bias, "router bias")
-    if score not in ("softmax", "chosen"):
-        raise KernelError(f"score `{score}` is not one of softmax, chosen")
+    _f32(shared_gate, "shared expert's gate")
+    if score not in _SCORES:
+        raise KernelError(f"score `{score}` is not one of {', '.join(_SCORES)}")
     _contig(h, "router input")
     _f32(router, "router matrix")
     _f32(correction, "router correction")
     n, W = h.shape
-    outputs = router.shape[0]
-    if router.shape != (outputs, W) or (correction is not None and correction.numel() != outputs) or \
+    outputs = router.shape[0] - (1 if shared_gate is not None else 0)
+    if shared_gate is not None and (shared_gate.numel() != n or outputs <= 0):
+        raise KernelError("the shared expert's gate is one number per token")
+    if router.shape[1] != W or (correction is not None and correction.numel() != outputs) or \
             (bias is not None and bias.numel() != outputs):
         raise KernelError("the router must be [outputs, W], the correction and the bias [outputs]")
     dev = h.device
@@ -1825,10 +1844,11 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.
         at += z
     ranks, offsets, pair_of, ntiles, tile_expert, tile_row0 = parts
     lib = _lib("moe")
-    _check(lib, lib.vapi_moe_route(_p(h), _dt(h), _p(router), _p(correction), _p(bias), 1 if score == "chosen" else 0,
+    _check(lib, lib.vapi_moe_route(_p(h), _dt(h), _p(router), _p(correction), _p(bias), _SCORES[score],
                                    _p(ids), _p(wts), _p(ranks),
                                    _p(offsets), _p(pair_of), _p(ntiles), _p(tile_expert), _p(tile_row0), n, W, outputs,
-                                   int(experts), int(top), int(groups), int(keep), _stream()), 2 if experts > 0 else 1)
+                                   int(experts), int(top), int(groups), int(keep), _stream(), int(group_top), _p(shared_gate)),
+           2 if experts > 0 else 1)
     return ids, wts, (offsets, pair_of, ntiles, tile_expert, tile_row0)
 
 
@@ -1863,15 +1883,17 @@ def moe_table_route(tokens: torch.Tensor, table: torch.Tensor, experts: int, sta
 
 def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, plan, w_up: Optional[torch.Tensor],
                 w_down: Optional[torch.Tensor], shared: Optional[torch.Tensor] = None, gated: bool = False,
-                act: Tuple[float, float, float] = (0.0, 1.0, 0.0)) -> torch.Tensor:
+                act: Tuple[float, float, float] = (0.0, 1.0, 0.0), shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The weighted sum of the chosen experts' outputs for ``h`` [n, W]: expert e is ``W_down[e] relu(W_up[e] h)^2``
     with ``w_up`` [experts, ff, W] and ``w_down`` [experts, W, ff] of h's dtype; a choice >= experts is an identity
-    expert (its output is h); ``shared`` [n, W] is added when given.  ``ids``, ``wts``, ``plan``: from
+    expert (its output is h); ``shared`` [n, W] is added when given, times ``shared_gate`` [n] float32 when that is
+    given too.  ``ids``, ``wts``, ``plan``: from
     :func:`moe_route`.  ``gated``: expert e is ``W_down[e] (silu(W_gate[e] h) * (W_up[e] h))`` and ``w_up`` is
     [experts, 2 * ff, W] with rows alternating gate_0, up_0, gate_1, up_1, ...  ``act`` = (limit, alpha, shift)
     generalises the gated form to ``g' * sigmoid(alpha g') * (u' + shift)`` with ``g' = min(g, limit)`` and
     ``u' = clamp(u, -limit, limit)`` when ``limit`` > 0 (the default is SiLU gating)."""
-    _cuda(h, ids, wts, w_up, w_down, shared)
+    _cuda(h, ids, wts, w_up, w_down, shared, shared_gate)
+    _f32(shared_gate, "shared expert's gate")
     limit, alpha, shift = (ctypes.c_float(float(v)) for v in act)
     _contig(h, "expert input")
     n, W = h.shape
@@ -1902,7 +1924,7 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, plan, w_u
             raise KernelError("the shared expert's output must have the input's shape and dtype")
     out = torch.empty_like(h)
     _check(lib, lib.vapi_moe_combine(_p(y), _p(ids), _p(wts), _p(h), _p(shared), _p(out), _dt(h), n, W, top, experts,
-                                     _stream()))
+                                     _stream(), _p(shared_gate)))
     return out
 
 
@@ -1973,4 +1995,53 @@ def gated_linear_attention(qkv: torch.Tensor, decay_logits: torch.Tensor, tau: f
         ctypes.c_longlong(decay_logits.stride(0)), ctypes.c_float(1.0 / tau), ctypes.c_float(q_scale), _p(state),
         ctypes.c_longlong(state.stride(0)), _p(state_slots), _p(cu_q), _p(positions), _p(out), n, cu_q.numel() - 1, nh, dk, dv,
         state.shape[0], int(min(max_q, 1 << 30)), _p(status), _stream()), 2 if max_q >= 16 else 1)
+    return out
+
+
+# ---------------------------------------------------------------------------------------
+# a decayed sum of outer products with a fixed decay per head (retention, lightning attention)
+#: tokens of a chunk of the chunked form (csrc/fixed_decay.cu)
+FIXED_DECAY_CHUNK = 128
+#: sequences that bring at least this many bfloat16 tokens take the chunked form on the tensor cores (0: never)
+FIXED_DECAY_CHUNK_MIN = int(os.environ.get("VAPI_FIXED_DECAY_CHUNK_MIN", "32"))
+
+
+def decay_powers(decay, device) -> torch.Tensor:
+    """``decay[h]^0 .. decay[h]^FIXED_DECAY_CHUNK`` as float32 [heads, FIXED_DECAY_CHUNK + 1], each rounded once from float64."""
+    d = torch.tensor([float(x) for x in decay], dtype=torch.float64)
+    i = torch.arange(FIXED_DECAY_CHUNK + 1, dtype=torch.float64)
+    return torch.pow(d[:, None], i[None, :]).to(torch.float32).to(device).contiguous()
+
+
+def fixed_decay_memory(qkv: torch.Tensor, powers: torch.Tensor, state: torch.Tensor, state_slots: torch.Tensor, cu_q: torch.Tensor,
+                       positions: torch.Tensor, nh: int, dk: int, dv: int, q_scale: float = 1.0, act: Optional[str] = None,
+                       status: Optional[torch.Tensor] = None, max_q: int = 1 << 30) -> torch.Tensor:
+    """Linear attention with one fixed decay per head over every sequence of the step: ``S <- decay_h S + k v^T;
+    o = q_scale * S^T q``.  ``qkv`` as for :func:`matrix_memory`; ``act`` "silu": q, k and v pass SiLU first.  ``powers``: from
+    :func:`decay_powers`.  ``state`` [slots, >= nh*dk*dv] float32 carries S [nh, dv, dk] (column by column).  Returns o
+    [n, nh*dv] float32.  Single tokens, short portions and float32 walk token by token; sequences that bring
+    ``FIXED_DECAY_CHUNK_MIN`` bfloat16 tokens or more are computed in chunks on the tensor cores (``max_q``: the most tokens
+    a sequence of the step brings)."""
+    _linear_memory_args(qkv, nh, dk, dv, state, nh * dk * dv, state_slots, cu_q, positions)
+    _cuda(powers)
+    if powers.dtype != torch.float32 or tuple(powers.shape) != (nh, FIXED_DECAY_CHUNK + 1) or not powers.is_contiguous():
+        raise KernelError(f"the decay's powers must be float32 [{nh}, {FIXED_DECAY_CHUNK + 1}] and contiguous")
+    if act not in (None, "silu"):
+        raise KernelError(f"activation `{act}` is not one of silu, None")
+    n, S = qkv.shape[0], cu_q.numel() - 1
+    max_q = int(min(max_q, n))
+    out = torch.empty((n, nh * dv), dtype=torch.float32, device=qkv.device)
+    lib = _lib("fixed_decay")
+    scratch, chunks, least = None, 0, FIXED_DECAY_CHUNK_MIN
+    if (0 < least <= max_q and qkv.dtype == torch.bfloat16 and dk % 8 == 0 and dv % 8 == 0 and qkv.stride(0) % 8 == 0
+            and qkv.data_ptr() % 16 == 0 and state.stride(0) % 2 == 0 and state.data_ptr() % 8 == 0):
+        chunks = n // FIXED_DECAY_CHUNK + min(S, n // least)
+        lib.vapi_fixed_decay_chunk_words.restype = ctypes.c_longlong
+        words = lib.vapi_fixed_decay_chunk_words(nh, dk, dv)
+        scratch = torch.empty((chunks * words * 4,), dtype=torch.int32, device=qkv.device)
+    launches = 1 if scratch is None else (2 if S == 1 else 3)
+    _check(lib, lib.vapi_fixed_decay(
+        _p(qkv), ctypes.c_longlong(qkv.stride(0)), 0, nh * dk, 2 * nh * dk, _dt(qkv), _p(powers), ctypes.c_float(q_scale),
+        1 if act == "silu" else 0, _p(state), ctypes.c_longlong(state.stride(0)), _p(state_slots), _p(cu_q), _p(positions), _p(out),
+        S, nh, dk, dv, state.shape[0], max_q, _p(scratch), chunks, int(least), _p(status), _stream()), launches)
     return out

@@ -15,7 +15,7 @@ from .latent import LatentAttention
 from .loop import StreamInjection
 from .hyper import HyperBlock, HyperPending
 from .parallel import ParallelMixer
-from .linear_memory import GatedLinearAttentionMixer, MatrixMemoryMixer
+from .linear_memory import FixedDecayMixer, GatedLinearAttentionMixer, MatrixMemoryMixer
 
 __all__ = [
     "CacheView", "FeedForward", "Mixer", "Norm", "NormedStream", "PagedBuffer", "PagedSpec", "StreamState", "Part", "PositionEncoding", "StateSpec",
@@ -25,5 +25,5 @@ __all__ = [
     "TokenEmbedding", "PreNormBlock", "SandwichBlock", "PostNormed", "ScaledRotaryEncoding", "GatedDeltaMixer", "Mamba2Mixer",
     "LayerNorm", "RGLRUMixer", "SparseMoE", "HyperBlock", "HyperPending", "ParallelMixer",
     "NoNorm", "MatrixMemoryMixer", "GatedLinearAttentionMixer", "ParallelBlock", "ScaledPair", "LatentAttention", "StreamInjection",
-    "ProjectedForm", "XIELU",
+    "ProjectedForm", "XIELU", "FixedDecayMixer",
 ]

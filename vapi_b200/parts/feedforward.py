@@ -13,11 +13,14 @@ class SwiGLU(FeedForward):
     """``down( silu(gate f) * (up f) )`` without biases; gate and up are stacked into one
     matrix at bind time so they are one product
     (crates/vapi-backend-candle/src/models/lfm2.rs:568-595).  ``names`` maps gate/up/down to
-    the checkpoint's sub-names (LFM2: w1 / w3 / w2).  ``bias``: ``down(silu(gate f + b_g) * (up f + b_u)) + b_d``."""
+    the checkpoint's sub-names (LFM2: w1 / w3 / w2).  ``bias``: ``down(silu(gate f + b_g) * (up f + b_u)) + b_d``.
+    ``act`` "gelu_tanh" puts the tanh form of GELU, ``0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))``, where SiLU stands."""
 
     def __init__(self, hidden: int, ff: int, names: Optional[Dict[str, str]] = None, weight_suffix: str = ".weight",
-                 bias: bool = False, bias_suffix: str = ".bias"):
-        self.hidden, self.ff, self.sfx = int(hidden), int(ff), weight_suffix
+                 bias: bool = False, bias_suffix: str = ".bias", act: str = "silu"):
+        if act not in ("silu", "gelu_tanh"):
+            raise ValueError(f"activation `{act}` is not one of silu, gelu_tanh")
+        self.hidden, self.ff, self.sfx, self.act = int(hidden), int(ff), weight_suffix, act
         #: with ``bias`` every projection adds a bias vector (``<name><bias_suffix>``)
         self.bias, self.bsfx = bool(bias), bias_suffix
         self.b_gate_up = self.b_down = None
@@ -49,8 +52,8 @@ class SwiGLU(FeedForward):
 
     def forward(self, f: torch.Tensor, ctx: Any) -> torch.Tensor:
         if self.bias:
-            return ops.linear(ops.swiglu(ops.linear(f, self.w_gate_up, self.b_gate_up)), self.w_down, self.b_down)
-        return ops.linear(ops.linear_swiglu(f, self.w_gate_up), self.w_down)
+            return ops.linear(ops.swiglu(ops.linear(f, self.w_gate_up, self.b_gate_up), act=self.act), self.w_down, self.b_down)
+        return ops.linear(ops.linear_swiglu(f, self.w_gate_up, act=self.act), self.w_down)
 
     def forward_stream(self, f, ctx, x, next_weight):
         if self.bias:
@@ -58,7 +61,7 @@ class SwiGLU(FeedForward):
         n = x.shape[0]
         if not (ops.few_rows_applies(n, self.w_gate_up) and ops.few_rows_applies(n, self.w_down)):
             return NotImplemented
-        s = ops.few_rows_linear(self.w_gate_up, xw=f.xw, ss_in=f.ss, eps=f.eps, epilogue="swiglu")
+        s = ops.few_rows_linear(self.w_gate_up, xw=f.xw, ss_in=f.ss, eps=f.eps, epilogue="swiglu", glu=self.act)
         ss, xw = ops.few_rows_linear(self.w_down, act=s, epilogue="resid", resid=x, next_weight=next_weight)
         return StreamState(xw, ss)
 

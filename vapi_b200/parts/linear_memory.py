@@ -1,15 +1,16 @@
 """Mixers whose state is a matrix per head that every token decays and adds an outer product to: the matrix
-memory of the xLSTM (mLSTM) and gated linear attention.
+memory of the xLSTM (mLSTM), gated linear attention, and linear attention with a fixed decay per head (retention,
+lightning attention).
 
-Both keep their matrices in the request's state slot as one float32 row, and their kernel
-(``csrc/linear_memory.cu``) walks each sequence of the step in order from the state that earlier steps left, so
-a prompt may be cut anywhere and a decode step is the same call with one token per sequence.  Gates, decays, their
+All keep their matrices in the request's state slot as one float32 row, and their kernels
+(``csrc/linear_memory.cu``, ``csrc/fixed_decay.cu``) take each sequence of the step in order from the state that earlier steps
+left, so a prompt may be cut anywhere and a decode step is the same call with one token per sequence.  Gates, decays, their
 logarithms and exponentials, the normalizer and the state are float32 whatever the activation dtype; the gates'
 pre-activations leave their products in float32.
 """
 from __future__ import annotations
 
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Sequence
 
 import torch
 
@@ -152,5 +153,70 @@ class GatedLinearAttentionMixer(Mixer):
         return ops.linear(y, self.w_o)
 
 
+class FixedDecayMixer(Mixer):
+    """Linear attention whose state decays by one fixed number per head: no softmax, no denominator.
+
+    ``q = act(W_q x)``, ``k = act(W_k x)`` (``n_heads`` of ``head_dim``), ``v = act(W_v x)`` (``n_heads`` of
+    ``v_head_dim``).  Per head ``S <- decay_h S + k v^T`` and ``o = qk_scale * S^T q``.  The heads' o are RMS-normed,
+    multiplied by a gate ``W_g x`` and projected by ``W_o``.  q, k, v and the gate are one product.
+
+    ``decay``: one number per head.  ``act``: "silu" or None.  ``norm``: "all" (over the concatenated heads together, with
+    a stored weight as wide) or "head" (each head by itself, no weight).  ``gate``: "sigmoid" or "silu".  ``qk_scale`` may
+    stand for a factor on q, on k, or on their product: the state holds k as it is and the read-out is multiplied.
+    """
+
+    def __init__(self, hidden: int, n_heads: int, head_dim: int, v_head_dim: int, decay: Sequence[float], norm_eps: float, *,
+                 act: Optional[str] = None, norm: str = "head", gate: str = "silu", qk_scale: float = 1.0,
+                 names: Optional[Dict[str, str]] = None, weight_suffix: str = ".weight"):
+        if n_heads <= 0 or not 1 <= head_dim <= 256 or v_head_dim <= 0:
+            raise ValueError(f"{n_heads} heads of {head_dim} x {v_head_dim} (keys up to 256)")
+        if len(decay) != n_heads:
+            raise ValueError(f"{len(decay)} decays for {n_heads} heads")
+        if act not in (None, "silu") or norm not in ("all", "head") or gate not in ("sigmoid", "silu"):
+            raise ValueError(f"activation `{act}`, norm `{norm}`, gate `{gate}`: one of silu or None; all, head; sigmoid, silu")
+        self.hidden, self.nh, self.dk, self.dv = int(hidden), int(n_heads), int(head_dim), int(v_head_dim)
+        self.decay = [float(d) for d in decay]
+        self.eps, self.act, self.norm, self.gate, self.qk_scale = float(norm_eps), act, norm, gate, float(qk_scale)
+        self.sfx = weight_suffix
+        self.names = {"q": "q_proj", "k": "k_proj", "v": "v_proj", "g": "g_proj", "o": "o_proj", "norm": "g_norm"}
+        if names:
+            self.names.update(names)
+        self.w_in = self.w_o = self.norm_w = self.powers = None
+
+    def cache_spec(self):
+        return StateSpec("fixed_decay", (self.nh * self.dk * self.dv,), torch.float32)
+
+    def tensor_specs(self, prefix: str) -> List[TensorSpec]:
+        n, h, x = self.names, self.hidden, self.sfx
+        qk, vv = self.nh * self.dk, self.nh * self.dv
+        specs = [TensorSpec(f"{prefix}{n['q']}{x}", (qk, h)), TensorSpec(f"{prefix}{n['k']}{x}", (qk, h)),
+                 TensorSpec(f"{prefix}{n['v']}{x}", (vv, h)), TensorSpec(f"{prefix}{n['g']}{x}", (vv, h)),
+                 TensorSpec(f"{prefix}{n['o']}{x}", (h, vv))]
+        if self.norm == "all":
+            specs.append(TensorSpec(f"{prefix}{n['norm']}", (vv,), role="vector", init="ones"))
+        return specs
+
+    def bind(self, tensors, prefix, dtype):
+        n, x = self.names, self.sfx
+        parts = [tensors[f"{prefix}{n[r]}{x}"] for r in ("q", "k", "v", "g")]
+        wd = parts[0].dtype if all(p.dtype == parts[0].dtype for p in parts) else torch.float32
+        self.w_in = torch.cat([p.to(wd) for p in parts], 0).contiguous()                  # q | k | v | g
+        self.w_o = tensors[f"{prefix}{n['o']}{x}"].contiguous()
+        self.norm_w = tensors[f"{prefix}{n['norm']}"].contiguous() if self.norm == "all" else \
+            torch.ones(self.dv, dtype=torch.float32, device=self.w_o.device)
+        self.powers = ops.decay_powers(self.decay, self.w_o.device)
+
+    def forward(self, a: torch.Tensor, ctx: Any, cache: CacheView) -> torch.Tensor:
+        nh, dk, dv = self.nh, self.dk, self.dv
+        h = ops.linear(a, self.w_in)
+        o = ops.fixed_decay_memory(h, self.powers, cache.tensor, ctx.state_slots, ctx.cu_q, ctx.positions, nh, dk, dv,
+                                   self.qk_scale, self.act, ctx.status, max_q=ctx.max_q)
+        off = 2 * nh * dk + nh * dv
+        y = ops.gated_group_rmsnorm(o, h[:, off:off + nh * dv], self.norm_w, self.eps, nh * dv if self.norm == "all" else dv,
+                                    False, h.dtype, gate=self.gate)
+        return ops.linear(y, self.w_o)
+
+
+register_mixer("fixed_decay", FixedDecayMixer)
 register_mixer("matrix_memory", MatrixMemoryMixer)
 register_mixer("gated_linear_attention", GatedLinearAttentionMixer)

@@ -25,7 +25,10 @@ class SparseMoE(FeedForward):
     ``route`` "table" (no router at all: a stored integer table [``vocab``, top] names the experts of each token id,
     each with weight ``1 / top``; the step's token ids choose) and, for gated experts, ``act`` = (limit, alpha,
     shift): ``g' * sigmoid(alpha g') * (u' + shift)`` with ``g' = min(W_gate f, limit)`` and
-    ``u' = clamp(W_up f, -limit, limit)`` when ``limit`` > 0 (the default (0, 1, 0) is SiLU gating).
+    ``u' = clamp(W_up f, -limit, limit)`` when ``limit`` > 0 (the default (0, 1, 0) is SiLU gating).  ``score`` "sigmoid": the
+    scores are the logits' sigmoids, one by one; ``correction`` False: no stored correction; ``group_top`` 2: a group's score
+    is the sum of its two largest; ``shared_gate``: the shared expert's output is multiplied by ``sigmoid(w_sg . f)``, one
+    number per token (w_sg rides on the router's product).
 
     The experts' matrices are stacked at bind time ([experts, ff, hidden] and [experts, hidden, ff]); a step's
     tokens are grouped by expert on the device (see ``csrc/moe.cu``), so nothing about the routing reaches the host.
@@ -34,7 +37,7 @@ class SparseMoE(FeedForward):
     def __init__(self, hidden: int, ff: int, experts: int, top: int, *, identity: int = 0, groups: int = 1, keep: int = 1,
                  shared_ff: Optional[int] = None, names: Optional[Dict[str, str]] = None, weight_suffix: str = ".weight",
                  gated: bool = False, router_bias: bool = False, score: str = "softmax", route: str = "router",
-                 vocab: int = 0, act=(0.0, 1.0, 0.0)):
+                 vocab: int = 0, act=(0.0, 1.0, 0.0), correction: bool = True, group_top: int = 1, shared_gate: bool = False):
         outputs = int(experts) + int(identity)
         if experts < 0 or identity < 0 or outputs <= 0 or not 1 <= top <= outputs:
             raise ValueError(f"{experts} experts + {identity} identity experts, top {top}")
@@ -42,8 +45,10 @@ class SparseMoE(FeedForward):
             raise ValueError(f"{outputs} router outputs in {groups} groups, {keep} kept, top {top}")
         self.hidden, self.ff, self.E, self.I, self.top = int(hidden), int(ff), int(experts), int(identity), int(top)
         self.groups, self.keep, self.shared_ff, self.sfx = int(groups), int(keep), shared_ff, weight_suffix
-        if score not in ("softmax", "chosen"):
-            raise ValueError(f"score `{score}` is not one of softmax, chosen")
+        if score not in ("softmax", "chosen", "sigmoid"):
+            raise ValueError(f"score `{score}` is not one of softmax, chosen, sigmoid")
+        if group_top not in (1, 2):
+            raise ValueError("a group's score comes from its largest one or two")
         if score == "chosen" and (groups != 1 or identity):
             raise ValueError("weights from the chosen logits come without groups and identity experts")
         if route not in ("router", "table"):
@@ -51,12 +56,17 @@ class SparseMoE(FeedForward):
         if route == "table" and (identity or groups != 1 or router_bias or vocab <= 0 or experts <= 0):
             raise ValueError("a table over the token ids chooses among real experts, without groups or a bias, and needs the vocabulary's size")
         self.by_table, self.vocab = route == "table", int(vocab)
+        if shared_gate and (shared_ff is None or self.by_table):
+            raise ValueError("a shared expert's gate needs a shared expert and a router")
+        self.group_top, self.gate_shared = int(group_top), bool(shared_gate)
+        self.corrected = bool(correction) and score != "chosen" and not self.by_table
         self.act = tuple(float(v) for v in act)
         if len(self.act) != 3 or (self.act != (0.0, 1.0, 0.0) and not gated):
             raise ValueError("the activation's constants (limit, alpha, shift) belong to gated experts")
         self.gated, self.router_bias, self.score = bool(gated), bool(router_bias), score
         self.names = {"expert": "experts.{}.", "up": "up_proj", "down": "down_proj", "gate": "gate_proj", "router": "router",
-                      "correction": "correction", "router_bias": "router.bias", "shared": "shared.", "table": "table"}
+                      "correction": "correction", "router_bias": "router.bias", "shared": "shared.", "table": "table",
+                      "shared_gate": "gate"}
         if names:
             self.names.update(names)
         self.router = self.correction = self.bias = self.w_up = self.w_down = self.s_up = self.s_down = self.s_gate = None
@@ -76,7 +86,7 @@ class SparseMoE(FeedForward):
         else:
             # the router works in float32 whatever the activation dtype
             specs.append(TensorSpec(f"{prefix}{n['router']}{x}", (self.E + self.I, h), role="vector"))
-        if self.score == "softmax" and not self.by_table:
+        if self.corrected:
             specs.append(TensorSpec(f"{prefix}{n['correction']}", (self.E + self.I,), role="vector", init="zeros"))
         if self.router_bias:
             specs.append(TensorSpec(f"{prefix}{n['router_bias']}", (self.E + self.I,), role="vector"))
@@ -85,6 +95,8 @@ class SparseMoE(FeedForward):
             if self.gated:
                 specs.append(TensorSpec(f"{sp}{n['gate']}{x}", (self.shared_ff, h)))
             specs += [TensorSpec(f"{sp}{n['up']}{x}", (self.shared_ff, h)), TensorSpec(f"{sp}{n['down']}{x}", (h, self.shared_ff))]
+            if self.gate_shared:
+                specs.append(TensorSpec(f"{sp}{n['shared_gate']}{x}", (1, h), role="vector"))
         return specs
 
     def bind(self, tensors, prefix, dtype):
@@ -102,7 +114,9 @@ class SparseMoE(FeedForward):
             self.table = tensors[f"{prefix}{n['table']}"].to(torch.int32).contiguous()
         else:
             self.router = tensors[f"{prefix}{n['router']}{x}"].contiguous()
-        self.correction = tensors[f"{prefix}{n['correction']}"].contiguous() if self.score == "softmax" and not self.by_table else None
+            if self.gate_shared:
+                self.router = torch.cat([self.router, tensors[f"{prefix}{n['shared']}{n['shared_gate']}{x}"]], 0).contiguous()
+        self.correction = tensors[f"{prefix}{n['correction']}"].contiguous() if self.corrected else None
         self.bias = tensors[f"{prefix}{n['router_bias']}"].contiguous() if self.router_bias else None
         if self.shared_ff is not None:
             sp = prefix + n["shared"]
@@ -113,17 +127,21 @@ class SparseMoE(FeedForward):
                 self.s_gate = torch.cat([g.to(self.s_up.dtype), self.s_up], 0).contiguous()      # gate | up, one product
 
     def forward(self, f: torch.Tensor, ctx: Any) -> torch.Tensor:
+        gate = None
         if self.by_table:
             ids, wts, plan = ops.moe_table_route(ctx.tokens, self.table, self.E, ctx.status)
         else:
+            if self.gate_shared:
+                gate = torch.empty((f.shape[0],), dtype=torch.float32, device=f.device)
             ids, wts, plan = ops.moe_route(f, self.router, self.correction, self.E, self.top, self.groups, self.keep,
-                                           bias=self.bias, score=self.score)
+                                           bias=self.bias, score=self.score, group_top=self.group_top, shared_gate=gate)
         shared = None
         if self.s_gate is not None:
             shared = ops.linear(ops.linear_swiglu(f, self.s_gate), self.s_down)
         elif self.s_up is not None:
             shared = ops.linear(ops.relu_squared(ops.linear(f, self.s_up)), self.s_down)
-        return ops.moe_experts(f, ids, wts, plan, self.w_up, self.w_down, shared, gated=self.gated, act=self.act)
+        return ops.moe_experts(f, ids, wts, plan, self.w_up, self.w_down, shared, gated=self.gated, act=self.act,
+                               shared_gate=gate)
 
 
 register_feed_forward("sparse_moe", SparseMoE)

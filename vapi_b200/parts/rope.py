@@ -41,9 +41,12 @@ class RotaryEncoding(PositionEncoding):
 
 
 class ScaledRotaryEncoding(PositionEncoding):
-    """Rotary tables whose frequencies an interpolation rule has changed (YaRN).
+    """Rotary tables whose frequencies an interpolation rule has changed (YaRN, or the rule of Llama 3.1).
 
-    ``f_i = base^(-2i / rot_dim)``.  With ``scaling = (factor, original, fast, slow)``: let
+    ``f_i = base^(-2i / rot_dim)``.  With ``scaling = (factor, original, low, high)``, by pair i's wavelength
+    ``l_i = 2 pi / f_i``: pairs of ``l_i < original / high`` keep ``f_i``, those of ``l_i > original / low`` turn at
+    ``f_i / factor``, and between the two ``s = (original / l_i - low) / (high - low)`` blends them,
+    ``(1 - s) f_i / factor + s f_i``.  With ``scaling = (factor, original, fast, slow)``: let
     ``c(t) = rot_dim * ln(original / (2 pi t)) / (2 ln base)`` (the pair index that makes ``t`` turns
     over ``original`` positions), ``lo = max(floor(c(fast)), 0)``, ``hi = min(ceil(c(slow)), rot_dim - 1)``
     and ``ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1)``; pair i then turns at
@@ -67,6 +70,19 @@ class ScaledRotaryEncoding(PositionEncoding):
         if not scaling:
             return f, 1.0
         factor, original = float(scaling["factor"]), float(scaling["original"])
+        if "low" in scaling:
+            low, high = float(scaling["low"]), float(scaling["high"])
+            out = []
+            for fi in f:
+                length = 2.0 * math.pi / fi
+                if length < original / high:
+                    out.append(fi)
+                elif length > original / low:
+                    out.append(fi / factor)
+                else:
+                    s = (original / length - low) / (high - low)
+                    out.append((1.0 - s) * fi / factor + s * fi)
+            return out, 1.0
 
         def pair_of(turns: float) -> float:
             return rot_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
