@@ -203,6 +203,7 @@ OPS = {"embed": "elementwise", "add_residual_ss": "elementwise", "resolve_tokens
        "embed_sinusoid": "hyper", "hyper_read_norm": "hyper", "branch_rmsnorm_mean": "hyper", "sigmoid_gate": "hyper",
        "softcap": "hyper", "causal_conv": "recurrent", "rglru": "rglru", "relu_squared": "moe", "moe_route": "moe",
        "moe_experts": "moe", "matrix_memory": "linear_memory", "gated_linear_attention": "linear_memory",
+       "fixed_decay_memory": "fixed_decay",
        "scaled_add_rmsnorm": "elementwise", "latent_prepare": "latent", "latent_rotate_q": "latent",
        "latent_attention": "attention_masked", "moe_table_route": "moe", "head_products": "library",
        "embed_bigram": "elementwise", "shift_add_rmsnorm": "elementwise", "xielu": "elementwise"}
@@ -863,10 +864,36 @@ def givavik_sizes(name):
     return gv, nelosun_sizes(name)[0], vukavik_sizes(name)[0]
 
 
+def zokelorn_sizes(name):
+    """Zokelorn layers at the widths of LFM2-<name>: lightning attention with heads of 128 x 128 across the width; retention
+    with heads of 128 x 256 (keys half as wide as the model in all, values as wide as it); attention with the same heads as
+    the LFM2 stack (keys and values of 64, chunks of 8,192, a gate per head, stretched frequencies); feed-forwards alternate
+    between a dense one of the LFM2 stack's width and a mixture of 32 experts (a quarter of that width each, four of them a
+    token, from two of four groups) with a gated shared expert of that quarter; eight layers in one pass of the loop.  Beside
+    it Demazen (matrix-state recurrences with the same states, gated experts behind a router, dense feed-forwards) and
+    Nelosun (attention on the same kernels, the same arrangement of a layer, gated experts) at the same widths."""
+    from vapi_b200.models.lfm2 import Lfm2Config
+    lf = lfm2_sizes(name)
+    W, ff = lf["hidden_size"], Lfm2Config.effective_ff_dim(lf)
+    dense = {"kind": "dense", "ff": ff}
+    sparse = {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 4},
+              "router": {"experts": 32, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    lin = {"heads": W // 128, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-1.0 - 8.0 * h * 128 / W) for h in range(W // 128)]}
+    ret = {"heads": W // 256, "dim": 128, "vdim": 256, "decay": [1.0 - 2.0 ** (-5.0 - h) for h in range(W // 256)]}
+    att = {"heads": lf["num_attention_heads"], "kv_heads": lf["num_key_value_heads"], "dim": 64, "vdim": 64, "scale": 0.125,
+           "mask": {"size": 8192}, "rot": {"base": 500000.0, "dims": 64,
+                                           "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    layers = [{"type": "lightning", "mixer": lin, "mlp": dense}, {"type": "retention", "mixer": ret, "mlp": sparse},
+              {"type": "lightning", "mixer": lin, "mlp": sparse}, {"type": "attention", "mixer": att, "mlp": dense}] * 2
+    zk = {"architecture": "Zokelorn", "vocab": lf["vocab_size"], "width": W, "norm": {"eps": 1e-5},
+          "loop": {"start": 0, "stop": 8, "times": 1}, "layers": layers}
+    return zk, demazen_sizes(name)[0], nelosun_sizes(name)[0]
+
+
 def mixers(args):
     """``--only mixers``: prefill and decode of eight layers of ``--design`` beside LFM2 layers (Vukavik, Rapolix; Demazen
     stands beside Vukavik and Rapolix, whose kernels are the nearest to its own, Nelosun beside Rapolix and Demazen, Givavik
-    beside Nelosun and Vukavik)
+    beside Nelosun and Vukavik, Zokelorn beside Demazen and Nelosun)
     of equal width (random weights), and where each model's time goes, kernel family by kernel family."""
     import torch
     from vapi_b200 import ops
@@ -890,6 +917,9 @@ def mixers(args):
     elif args.design == "givavik":
         gv, ne, vk = givavik_sizes(args.sizes)
         models = (("givavik", gv), ("nelosun", ne), ("vukavik", vk))
+    elif args.design == "zokelorn":
+        zk, dz, ne = zokelorn_sizes(args.sizes)
+        models = (("zokelorn", zk), ("demazen", dz), ("nelosun", ne))
     else:
         vk, lf = rapolix_sizes(args.sizes) if args.design == "rapolix" else vukavik_sizes(args.sizes)
         models = ((args.design, vk), ("lfm2", lf))
@@ -959,6 +989,10 @@ def mixers(args):
                 mix_flops["state_space"] = 2.0 * 3 * m.nh * m.N * m.p * T        # decay, the rank-one write, S^T C
             elif kind == "MatrixMemoryMixer":
                 mix_flops["matrix_memory"] = 2.0 * 3 * m.nh * m.dk * m.dv * T    # decay, the rank-one write, S^T q
+            elif kind == "FixedDecayMixer":
+                # (per call, of the token-by-token form; layers of two kinds: their mean)
+                mix_flops.setdefault("fixed_decay_each", []).append(2.0 * 3 * m.nh * m.dk * m.dv * T)
+                mix_flops["fixed_decay_memory"] = sum(mix_flops["fixed_decay_each"]) / len(mix_flops["fixed_decay_each"])
             elif kind == "GatedLinearAttentionMixer":
                 mix_flops["gated_linear_attention"] = 2.0 * 3 * m.nh * m.dk * m.dv * T
         rows = {}
@@ -1061,9 +1095,10 @@ def main():
                          "and print what one step's kernels did inside the captured graph, or (mixers) prefill and "
                          "decode of eight Vukavik layers beside eight LFM2 layers of equal width, kernel family by kernel family")
     ap.add_argument("--sizes", default="1.2b", choices=["1.2b", "700m", "2.6b"], help="layer sizes of LFM2-<sizes>")
-    ap.add_argument("--design", default="vukavik", choices=["vukavik", "rapolix", "demazen", "nelosun", "givavik"],
+    ap.add_argument("--design", default="vukavik", choices=["vukavik", "rapolix", "demazen", "nelosun", "givavik", "zokelorn"],
                     help="with --only mixers: the architecture whose layers stand beside LFM2's (demazen: beside Vukavik's and "
-                         "Rapolix's; nelosun: beside Rapolix's and Demazen's; givavik: beside Nelosun's and Vukavik's)")
+                         "Rapolix's; nelosun: beside Rapolix's and Demazen's; givavik: beside Nelosun's and Vukavik's; "
+                         "zokelorn: beside Demazen's and Nelosun's)")
     ap.add_argument("--page-size", type=int, default=0, help="tokens per cache page (0: the engine's default)")
     ap.add_argument("--dtype", default="bfloat16", help="bfloat16 (serving) or float32 (the true 32-bit path)")
     ap.add_argument("--no-fp32", action="store_true", help="leave the float32 points out of the default run")

@@ -118,16 +118,17 @@ def prompt(cfg: dict, n: int, seed: int):
 
 class Oracle:
     """The plain model on a folder, float64."""
+    model = plain
 
     def __init__(self, folder: str):
-        self.cfg = plain.read_config(folder)
-        self.w = plain.read_weights(folder, torch.float64)
+        self.cfg = self.model.read_config(folder)
+        self.w = self.model.read_weights(folder, torch.float64)
         self._memo: Dict[tuple, object] = {}
 
     def logits(self, tokens: Sequence[int]) -> torch.Tensor:
         key = tuple(tokens)
         if key not in self._memo:
-            self._memo[key] = plain.forward(self.cfg, self.w, tokens)
+            self._memo[key] = self.model.forward(self.cfg, self.w, tokens)
         return self._memo[key]
 
     def rounding(self, tokens: Sequence[int], dtype: str = "float32") -> np.ndarray:
@@ -144,9 +145,9 @@ class Oracle:
                 return {k: (v * (1.0 + by * (2.0 * torch.rand(v.shape, generator=g, dtype=v.dtype) - 1.0))).to(to)
                         if v.dim() >= 2 or to == torch.float32 else v for k, v in self.w.items()}
             if dtype == "float32":
-                draws = [plain.forward(self.cfg, moved(by, torch.float32), tokens).double() for by in (0.0, 2.0 ** -23)]
+                draws = [self.model.forward(self.cfg, moved(by, torch.float32), tokens).double() for by in (0.0, 2.0 ** -23)]
             else:
-                draws = [plain.forward(self.cfg, moved(2.0 ** -8, torch.float64), tokens)]
+                draws = [self.model.forward(self.cfg, moved(2.0 ** -8, torch.float64), tokens)]
             err = torch.stack([(got - want).abs().amax(-1) for got in draws]).amax(0)
             self._memo[key] = (err / float(want.max() - want.min())).numpy()
         return self._memo[key]
