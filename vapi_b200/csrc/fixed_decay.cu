@@ -217,8 +217,9 @@ fixed_decay_walk_kernel(const T* __restrict__ qkv, long long qkv_stride, int q_o
 }
 
 // ---- chunks ----------------------------------------------------------------------------------------------
-constexpr int FD_CB = 64;          // columns of S a block of the first kernel owns (16 a warp); of the second too
-constexpr int FD_RB = 32;          // rows of S a block of the first kernel owns
+constexpr int FD_CT = 256;         // threads of a block of either kernel
+constexpr int FD_CB = 64;          // columns of S a block of the first kernel owns; of the second too
+constexpr int FD_RB = 32;          // rows of S a block of the first kernel owns (a warp: 16 columns x 16 rows)
 constexpr int FD_VLD = FD_CB + 8, FD_KLD = FD_RB + 8;       // shared rows end 16 bytes further: ldmatrix without bank conflicts
 
 // eight bfloat16 numbers, through SiLU when asked for
@@ -258,8 +259,8 @@ __device__ __forceinline__ int fd_chunks_before(const int* __restrict__ cu_q, in
 }
 
 // Walks the chunks of one (sequence, head) for a part of S (FD_CB columns x FD_RB rows).  A warp's accumulators are S^T:
-// 16 columns x 32 rows, in four tiles of eight rows.
-__global__ void __launch_bounds__(FD_THREADS)
+// 16 columns x 16 rows, in two tiles of eight rows.
+__global__ void __launch_bounds__(FD_CT)
 fixed_decay_states_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_stride, int k_off, int v_off,
                           const float* __restrict__ powers, int act, float* __restrict__ state, long long slot_stride,
                           const int* __restrict__ state_slots, const int* __restrict__ cu_q, const int* __restrict__ positions,
@@ -267,11 +268,11 @@ fixed_decay_states_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_s
                           int* __restrict__ status) {
     __shared__ __align__(16) __nv_bfloat16 sV[FD_C * FD_VLD], sKh[FD_C * FD_KLD], sKl[FD_C * FD_KLD];
     __shared__ float pw[FD_C + 1];
-    constexpr int VP = FD_C * FD_CB / 8 / FD_THREADS, KP = FD_C * FD_RB / 8 / FD_THREADS;      // 16-byte pieces a thread brings
+    constexpr int VP = FD_C * FD_CB / 8 / FD_CT, KP = FD_C * FD_RB / 8 / FD_CT;      // 16-byte pieces a thread brings
     const int s = blockIdx.z, h = blockIdx.y;
     const int rblocks = (rows + FD_RB - 1) / FD_RB;
     const int col0 = (blockIdx.x / rblocks) * FD_CB, row0 = (blockIdx.x % rblocks) * FD_RB;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int wc = (threadIdx.x >> 5) & 3, wr = threadIdx.x >> 7, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int t0 = cu_q[s], qlen = cu_q[s + 1] - t0;
     if (qlen < min_q) return;
     const int slot = state_slots[s];
@@ -281,17 +282,17 @@ fixed_decay_states_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_s
         if (threadIdx.x == 0 && status) atomicExch(status, 3);
         return;
     }
-    for (int i = threadIdx.x; i <= FD_C; i += FD_THREADS) pw[i] = powers[(size_t)h * (FD_C + 1) + i];
+    for (int i = threadIdx.x; i <= FD_C; i += FD_CT) pw[i] = powers[(size_t)h * (FD_C + 1) + i];
     const int KS = (rows + 15) / 16, CT = (cols + 7) / 8;
     pdl_wait();
     const bool fresh = positions[t0] == 0;
 
-    float acc[4][4];
+    float acc[2][4];
     float* S_glob = state + (size_t)slot * slot_stride + (size_t)h * cols * rows;
-    const int ca = col0 + warp * 16 + g;                      // this lane's columns: ca and ca + 8
+    const int ca = col0 + wc * 16 + g;                      // this lane's columns: ca and ca + 8
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt) {
-        const int r = row0 + nt * 8 + 2 * t;
+    for (int nt = 0; nt < 2; ++nt) {
+        const int r = row0 + wr * 16 + nt * 8 + 2 * t;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             const int c = ca + 8 * half;
@@ -309,12 +310,12 @@ fixed_decay_states_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_s
         const __nv_bfloat16* at = qkv + (size_t)(t0 + first) * qkv_stride;
 #pragma unroll
         for (int i = 0; i < VP; ++i) {
-            const int idx = threadIdx.x + i * FD_THREADS, tok = idx / (FD_CB / 8), cc = col0 + (idx % (FD_CB / 8)) * 8;
+            const int idx = threadIdx.x + i * FD_CT, tok = idx / (FD_CB / 8), cc = col0 + (idx % (FD_CB / 8)) * 8;
             rv[i] = tok < L && cc < cols ? *reinterpret_cast<const uint4*>(at + (size_t)tok * qkv_stride + v_off + (size_t)h * cols + cc) : zero;
         }
 #pragma unroll
         for (int i = 0; i < KP; ++i) {
-            const int idx = threadIdx.x + i * FD_THREADS, tok = idx / (FD_RB / 8), rr = row0 + (idx % (FD_RB / 8)) * 8;
+            const int idx = threadIdx.x + i * FD_CT, tok = idx / (FD_RB / 8), rr = row0 + (idx % (FD_RB / 8)) * 8;
             rk[i] = tok < L && rr < rows ? *reinterpret_cast<const uint4*>(at + (size_t)tok * qkv_stride + k_off + (size_t)h * rows + rr) : zero;
         }
     };
@@ -325,12 +326,12 @@ fixed_decay_states_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_s
         __syncthreads();                                      // the products of the chunk before have read shared memory
 #pragma unroll
         for (int i = 0; i < VP; ++i) {
-            const int idx = threadIdx.x + i * FD_THREADS, tok = idx / (FD_CB / 8), piece = idx % (FD_CB / 8);
+            const int idx = threadIdx.x + i * FD_CT, tok = idx / (FD_CB / 8), piece = idx % (FD_CB / 8);
             *reinterpret_cast<uint4*>(sV + tok * FD_VLD + piece * 8) = fd_act8(rv[i], act);
         }
 #pragma unroll
         for (int i = 0; i < KP; ++i) {
-            const int idx = threadIdx.x + i * FD_THREADS, tok = idx / (FD_RB / 8), piece = idx % (FD_RB / 8);
+            const int idx = threadIdx.x + i * FD_CT, tok = idx / (FD_RB / 8), piece = idx % (FD_RB / 8);
             const float p = pw[max(L - 1 - tok, 0)];          // (tokens behind the chunk are rows of zeros)
             float f[8];
             fd_unpack8(rk[i], f, act);
@@ -348,45 +349,38 @@ fixed_decay_states_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_s
             uint4* dst = scratch + ((size_t)(base + c) * nh + h) * ((size_t)KS * CT * 32);
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
-                const int ct = (col0 + warp * 16) / 8 + half;
-#pragma unroll
-                for (int kk = 0; kk < 2; ++kk) {
-                    const int ks = row0 / 16 + kk;
-                    if (ct < CT && ks < KS) {
-                        uint4 w;
-                        fd_split(acc[2 * kk][2 * half], acc[2 * kk][2 * half + 1], w.x, w.z);
-                        fd_split(acc[2 * kk + 1][2 * half], acc[2 * kk + 1][2 * half + 1], w.y, w.w);
-                        dst[((size_t)ct * KS + ks) * 32 + lane] = w;
-                    }
+                const int ct = (col0 + wc * 16) / 8 + half, ks = row0 / 16 + wr;
+                if (ct < CT && ks < KS) {
+                    uint4 w;
+                    fd_split(acc[0][2 * half], acc[0][2 * half + 1], w.x, w.z);
+                    fd_split(acc[1][2 * half], acc[1][2 * half + 1], w.y, w.w);
+                    dst[((size_t)ct * KS + ks) * 32 + lane] = w;
                 }
             }
         }
         const float pl = pw[L];
 #pragma unroll
-        for (int nt = 0; nt < 4; ++nt)
+        for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
             for (int i = 0; i < 4; ++i) acc[nt][i] *= pl;
         const int ksteps = (L + 15) / 16;
-#pragma unroll 2
+#pragma unroll 4
         for (int kt = 0; kt < ksteps; ++kt) {
             unsigned a[4];
-            ldmatrix_x4_trans(a[0], a[1], a[2], a[3], sV + (kt * 16 + (mat >> 1) * 8 + rin) * FD_VLD + warp * 16 + (mat & 1) * 8);
-#pragma unroll
-            for (int nn = 0; nn < 2; ++nn) {
-                const int at = (kt * 16 + (mat & 1) * 8 + rin) * FD_KLD + nn * 16 + (mat >> 1) * 8;
-                unsigned b0, b1, b2, b3;
-                ldmatrix_x4_trans(b0, b1, b2, b3, sKh + at);
-                mma_bf16_16816(acc[2 * nn], a, b0, b1);
-                mma_bf16_16816(acc[2 * nn + 1], a, b2, b3);
-                ldmatrix_x4_trans(b0, b1, b2, b3, sKl + at);
-                mma_bf16_16816(acc[2 * nn], a, b0, b1);
-                mma_bf16_16816(acc[2 * nn + 1], a, b2, b3);
-            }
+            ldmatrix_x4_trans(a[0], a[1], a[2], a[3], sV + (kt * 16 + (mat >> 1) * 8 + rin) * FD_VLD + wc * 16 + (mat & 1) * 8);
+            const int at = (kt * 16 + (mat & 1) * 8 + rin) * FD_KLD + wr * 16 + (mat >> 1) * 8;
+            unsigned b0, b1, b2, b3;
+            ldmatrix_x4_trans(b0, b1, b2, b3, sKh + at);
+            mma_bf16_16816(acc[0], a, b0, b1);
+            mma_bf16_16816(acc[1], a, b2, b3);
+            ldmatrix_x4_trans(b0, b1, b2, b3, sKl + at);
+            mma_bf16_16816(acc[0], a, b0, b1);
+            mma_bf16_16816(acc[1], a, b2, b3);
         }
     }
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt) {
-        const int r = row0 + nt * 8 + 2 * t;
+    for (int nt = 0; nt < 2; ++nt) {
+        const int r = row0 + wr * 16 + nt * 8 + 2 * t;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             const int c = ca + 8 * half;
@@ -395,9 +389,9 @@ fixed_decay_states_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_s
     }
 }
 
-// One chunk of one (sequence, head), FD_CB columns of the output.  A warp owns two tiles of 16 tokens, the w-th and
-// the w-th from the end, so that all warps meet the same number of earlier tokens.
-__global__ void __launch_bounds__(FD_THREADS)
+// One chunk of one (sequence, head), FD_CB columns of the output.  A warp owns 16 tokens; which 16 is arranged so that
+// the two warps of a scheduler together meet the same number of earlier tokens as any other two.
+__global__ void __launch_bounds__(FD_CT, 2)
 fixed_decay_output_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_stride, int q_off, int k_off, int v_off,
                           const float* __restrict__ powers, float q_scale, int act, const int* __restrict__ state_slots,
                           const int* __restrict__ cu_q, const int* __restrict__ positions, const uint4* __restrict__ scratch,
@@ -419,134 +413,128 @@ fixed_decay_output_kernel(const __nv_bfloat16* __restrict__ qkv, long long qkv_s
     const int base = fd_chunks_before(cu_q, s, min_q);
     if (slot < 0 || slot >= num_slots || base + (qlen + FD_C - 1) / FD_C > scratch_chunks) return;     // (the first kernel has said so)
     const int L = min(FD_C, qlen - c * FD_C);
-    for (int i = threadIdx.x; i <= FD_C; i += FD_THREADS) pw[i] = powers[(size_t)h * (FD_C + 1) + i];
+    for (int i = threadIdx.x; i <= FD_C; i += FD_CT) pw[i] = powers[(size_t)h * (FD_C + 1) + i];
     pdl_wait();
     const bool has_state = c > 0 || positions[t0] != 0;
     const __nv_bfloat16* at = qkv + (size_t)(t0 + c * FD_C) * qkv_stride;
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
     const int pieces = KS * 2;                                // 16-byte pieces of a row of q or k
     const int LT = (L + 15) & ~15;                            // rows that the tiles read
-#pragma unroll 4
-    for (int idx = threadIdx.x; idx < LT * pieces; idx += FD_THREADS) {
-        const int tok = idx / pieces, r = (idx - tok * pieces) * 8;
-        const bool ok = tok < L && r < rows;
-        const __nv_bfloat16* p = at + (size_t)tok * qkv_stride + (size_t)h * rows + r;
-        const uint4 qv = ok ? *reinterpret_cast<const uint4*>(p + q_off) : zero;
-        const uint4 kv = ok ? *reinterpret_cast<const uint4*>(p + k_off) : zero;
-        *reinterpret_cast<uint4*>(sQ + tok * ld + r) = fd_act8(qv, act);
-        *reinterpret_cast<uint4*>(sK + tok * ld + r) = fd_act8(kv, act);
+    constexpr int IN = 4;                                     // pieces of q and of k a thread has in flight
+    for (int i0 = 0; i0 < LT * pieces; i0 += IN * FD_CT) {
+        uint4 qv[IN], kv[IN];
+        int to[IN];
+#pragma unroll
+        for (int i = 0; i < IN; ++i) {
+            const int idx = i0 + i * FD_CT + threadIdx.x;
+            const int tok = idx / pieces, r = (idx - tok * pieces) * 8;
+            const bool ok = tok < L && r < rows;
+            const __nv_bfloat16* p = at + (size_t)tok * qkv_stride + (size_t)h * rows + r;
+            qv[i] = ok ? *reinterpret_cast<const uint4*>(p + q_off) : zero;
+            kv[i] = ok ? *reinterpret_cast<const uint4*>(p + k_off) : zero;
+            to[i] = tok < LT ? tok * ld + r : -1;
+        }
+#pragma unroll
+        for (int i = 0; i < IN; ++i) {
+            if (to[i] < 0) continue;
+            *reinterpret_cast<uint4*>(sQ + to[i]) = fd_act8(qv[i], act);
+            *reinterpret_cast<uint4*>(sK + to[i]) = fd_act8(kv[i], act);
+        }
     }
-#pragma unroll 4
-    for (int idx = threadIdx.x; idx < LT * (FD_CB / 8); idx += FD_THREADS) {
-        const int tok = idx / (FD_CB / 8), cc = (idx % (FD_CB / 8)) * 8;
+#pragma unroll
+    for (int i = 0; i < FD_C * FD_CB / 8 / FD_CT; ++i) {
+        const int idx = threadIdx.x + i * FD_CT, tok = idx / (FD_CB / 8), cc = (idx % (FD_CB / 8)) * 8;
         const uint4 vv = tok < L && col0 + cc < cols ? *reinterpret_cast<const uint4*>(at + (size_t)tok * qkv_stride + v_off + (size_t)h * cols + col0 + cc) : zero;
         *reinterpret_cast<uint4*>(sV + tok * FD_VLD + cc) = fd_act8(vv, act);
     }
-    __syncthreads();
-    const int tiles = LT / 16;
-    const int mt[2] = {warp, FD_C / 16 - 1 - warp};
-    const bool on[2] = {mt[0] < tiles, mt[1] < tiles};
-    if (!on[0]) return;                                       // (the first of a warp's tiles is the earlier one)
+    const int mt = warp < 4 ? warp : 11 - warp;               // (warps w and w + 4 share a scheduler)
+    const bool on = mt * 16 < LT;
     const int mat = lane >> 3, rin = lane & 7;
-    float o[2][8][4];
+    // the state's first operands are on their way while the others finish loading
+    const uint4* src = scratch + ((size_t)(base + c) * nh + h) * ((size_t)KS * CT * 32) + lane;
+    const int ct0 = col0 / 8;
+    uint4 f[8];
+    auto load_s = [&](int ks) {
 #pragma unroll
-    for (int m = 0; m < 2; ++m)
-#pragma unroll
-        for (int n = 0; n < 8; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f;
-    auto load_q = [&](int m, int ks, unsigned (&a)[4]) {
-        ldmatrix_x4(a[0], a[1], a[2], a[3], sQ + (mt[m] * 16 + (mat & 1) * 8 + rin) * ld + ks * 16 + (mat >> 1) * 8);
+        for (int n = 0; n < 8; ++n) f[n] = ct0 + n < CT ? src[((size_t)(ct0 + n) * KS + ks) * 32] : zero;
     };
-    if (has_state) {
-        const uint4* src = scratch + ((size_t)(base + c) * nh + h) * ((size_t)KS * CT * 32) + lane;
-        const int ct0 = col0 / 8;
-        uint4 f[8];
-        auto load_s = [&](int ks) {
+    if (has_state && on) load_s(0);
+    __syncthreads();
+    if (!on) return;
+    float o[8][4];
 #pragma unroll
-            for (int n = 0; n < 8; ++n) f[n] = ct0 + n < CT ? src[((size_t)(ct0 + n) * KS + ks) * 32] : zero;
-        };
-        load_s(0);
+    for (int n = 0; n < 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+    const __nv_bfloat16* q_mine = sQ + (mt * 16 + (mat & 1) * 8 + rin) * ld + (mat >> 1) * 8;
+    if (has_state) {
         for (int ks = 0; ks < KS; ++ks) {
             uint4 w[8];
 #pragma unroll
             for (int n = 0; n < 8; ++n) w[n] = f[n];
             if (ks + 1 < KS) load_s(ks + 1);
+            unsigned a[4];
+            ldmatrix_x4(a[0], a[1], a[2], a[3], q_mine + ks * 16);
 #pragma unroll
-            for (int m = 0; m < 2; ++m) {
-                if (!on[m]) continue;
-                unsigned a[4];
-                load_q(m, ks, a);
+            for (int n = 0; n < 8; ++n) mma_bf16_16816(o[n], a, w[n].x, w[n].y);
 #pragma unroll
-                for (int n = 0; n < 8; ++n) {
-                    mma_bf16_16816(o[m][n], a, w[n].x, w[n].y);
-                    mma_bf16_16816(o[m][n], a, w[n].z, w[n].w);
-                }
-            }
+            for (int n = 0; n < 8; ++n) mma_bf16_16816(o[n], a, w[n].z, w[n].w);
         }
+        const float pa = pw[mt * 16 + g + 1], pb = pw[mt * 16 + g + 9];
 #pragma unroll
-        for (int m = 0; m < 2; ++m) {
-            const float pa = pw[mt[m] * 16 + g + 1], pb = pw[mt[m] * 16 + g + 9];
-#pragma unroll
-            for (int n = 0; n < 8; ++n) { o[m][n][0] *= pa; o[m][n][1] *= pa; o[m][n][2] *= pb; o[m][n][3] *= pb; }
-        }
+        for (int n = 0; n < 8; ++n) { o[n][0] *= pa; o[n][1] *= pa; o[n][2] *= pb; o[n][3] *= pb; }
     }
-    const int last = on[1] ? mt[1] : mt[0];
-    for (int jb = 0; jb <= last; ++jb) {                      // sixteen earlier tokens at a time
-        const bool here[2] = {jb <= mt[0], on[1]};
+    for (int jb = 0; jb <= mt; ++jb) {                        // sixteen earlier tokens at a time
+        // (even and odd steps of the inner size add up apart: two chains instead of one)
         float a[2][2][4];
 #pragma unroll
-        for (int m = 0; m < 2; ++m)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
-            for (int n = 0; n < 2; ++n) a[m][n][0] = a[m][n][1] = a[m][n][2] = a[m][n][3] = 0.f;
-#pragma unroll 2
-        for (int ks = 0; ks < KS; ++ks) {
-            unsigned b0, b1, b2, b3;
-            ldmatrix_x4(b0, b1, b2, b3, sK + (jb * 16 + (mat >> 1) * 8 + rin) * ld + ks * 16 + (mat & 1) * 8);
+            for (int e = 0; e < 4; ++e) a[0][n][e] = a[1][n][e] = 0.f;
+        const __nv_bfloat16* k_mine = sK + (jb * 16 + (mat >> 1) * 8 + rin) * ld + (mat & 1) * 8;
+        for (int ks = 0; ks < KS; ks += 2) {
 #pragma unroll
-            for (int m = 0; m < 2; ++m) {
-                if (!here[m]) continue;
-                unsigned q[4];
-                load_q(m, ks, q);
-                mma_bf16_16816(a[m][0], q, b0, b1);
-                mma_bf16_16816(a[m][1], q, b2, b3);
+            for (int x = 0; x < 2; ++x) {
+                if (ks + x >= KS) break;
+                unsigned q[4], b0, b1, b2, b3;
+                ldmatrix_x4(q[0], q[1], q[2], q[3], q_mine + (ks + x) * 16);
+                ldmatrix_x4(b0, b1, b2, b3, k_mine + (ks + x) * 16);
+                mma_bf16_16816(a[x][0], q, b0, b1);
+                mma_bf16_16816(a[x][1], q, b2, b3);
             }
         }
-        unsigned hi[2][4], lo[2][4];
+        unsigned hi[4], lo[4];
 #pragma unroll
-        for (int m = 0; m < 2; ++m)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
-            for (int n = 0; n < 2; ++n)
+            for (int e = 0; e < 2; ++e) {                     // rows g and g + 8 of the tile
+                const int d = mt * 16 + g + 8 * e - (jb * 16 + n * 8 + 2 * t);              // how far back the first of the pair lies
+                const float x = d >= 0 ? (a[0][n][2 * e] + a[1][n][2 * e]) * pw[max(d, 0)] : 0.f;
+                const float y = d >= 1 ? (a[0][n][2 * e + 1] + a[1][n][2 * e + 1]) * pw[max(d - 1, 0)] : 0.f;
+                fd_split(x, y, hi[2 * n + e], lo[2 * n + e]);
+            }
+        unsigned b[4][4];
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {                 // rows g and g + 8 of the tile
-                    const int d = mt[m] * 16 + g + 8 * e - (jb * 16 + n * 8 + 2 * t);       // how far back the first of the pair lies
-                    const float x = d >= 0 ? a[m][n][2 * e] * pw[max(d, 0)] : 0.f;
-                    const float y = d >= 1 ? a[m][n][2 * e + 1] * pw[max(d - 1, 0)] : 0.f;
-                    fd_split(x, y, hi[m][2 * n + e], lo[m][2 * n + e]);
-                }
+        for (int nn = 0; nn < 4; ++nn)
+            ldmatrix_x4_trans(b[nn][0], b[nn][1], b[nn][2], b[nn][3], sV + (jb * 16 + (mat & 1) * 8 + rin) * FD_VLD + nn * 16 + (mat >> 1) * 8);
 #pragma unroll
         for (int nn = 0; nn < 4; ++nn) {
-            unsigned b0, b1, b2, b3;
-            ldmatrix_x4_trans(b0, b1, b2, b3, sV + (jb * 16 + (mat & 1) * 8 + rin) * FD_VLD + nn * 16 + (mat >> 1) * 8);
+            mma_bf16_16816(o[2 * nn], hi, b[nn][0], b[nn][1]);
+            mma_bf16_16816(o[2 * nn + 1], hi, b[nn][2], b[nn][3]);
+        }
 #pragma unroll
-            for (int m = 0; m < 2; ++m) {
-                if (!here[m]) continue;
-                mma_bf16_16816(o[m][2 * nn], hi[m], b0, b1);
-                mma_bf16_16816(o[m][2 * nn + 1], hi[m], b2, b3);
-                mma_bf16_16816(o[m][2 * nn], lo[m], b0, b1);
-                mma_bf16_16816(o[m][2 * nn + 1], lo[m], b2, b3);
-            }
+        for (int nn = 0; nn < 4; ++nn) {
+            mma_bf16_16816(o[2 * nn], lo, b[nn][0], b[nn][1]);
+            mma_bf16_16816(o[2 * nn + 1], lo, b[nn][2], b[nn][3]);
         }
     }
 #pragma unroll
-    for (int m = 0; m < 2; ++m)
+    for (int e = 0; e < 2; ++e) {
+        const int i = mt * 16 + g + 8 * e;
+        if (i >= L) continue;
+        float* row = out + ((size_t)(t0 + c * FD_C + i) * nh + h) * cols + col0 + 2 * t;
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const int i = mt[m] * 16 + g + 8 * e;
-            if (i >= L) continue;
-            float* row = out + ((size_t)(t0 + c * FD_C + i) * nh + h) * cols + col0 + 2 * t;
-#pragma unroll
-            for (int n = 0; n < 8; ++n)
-                if (col0 + n * 8 < cols) *reinterpret_cast<float2*>(row + n * 8) = make_float2(q_scale * o[m][n][2 * e], q_scale * o[m][n][2 * e + 1]);
-        }
+        for (int n = 0; n < 8; ++n)
+            if (col0 + n * 8 < cols) *reinterpret_cast<float2*>(row + n * 8) = make_float2(q_scale * o[n][2 * e], q_scale * o[n][2 * e + 1]);
+    }
 }
 
 VAPI_EXPORT int vapi_fixed_decay_chunk() { return FD_C; }
@@ -578,7 +566,7 @@ VAPI_EXPORT int vapi_fixed_decay(const void* qkv, long long qkv_stride, int q_of
             slot_stride % 2 || ((uintptr_t)state & 7) || ((uintptr_t)out & 7))
             return fail(-1, "fixed_decay: the chunked form needs 16-byte aligned rows");
         dim3 grid(((cols + FD_CB - 1) / FD_CB) * ((rows + FD_RB - 1) / FD_RB), nh, num_seqs);
-        cudaError_t e = launch_if(false, fixed_decay_states_kernel, grid, FD_THREADS, 0, stream, (const __nv_bfloat16*)qkv, qkv_stride,
+        cudaError_t e = launch_if(false, fixed_decay_states_kernel, grid, FD_CT, 0, stream, (const __nv_bfloat16*)qkv, qkv_stride,
                                   k_off, v_off, powers, act, state, slot_stride, state_slots, cu_q, positions, (uint4*)scratch,
                                   scratch_chunks, nh, rows, cols, num_slots, min_q, status);
         int rc = check_launch("fixed_decay (states)", e);
@@ -593,7 +581,7 @@ VAPI_EXPORT int vapi_fixed_decay(const void* qkv, long long qkv_stride, int q_of
         }
         const long long bx = (long long)((max_q + FD_C - 1) / FD_C) * ((cols + FD_CB - 1) / FD_CB);
         if (bx > 0x7fffffffLL) return fail(-1, "fixed_decay: %d tokens are too many", max_q);
-        e = launch(fixed_decay_output_kernel, dim3((unsigned)bx, nh, num_seqs), FD_THREADS, smem, stream, (const __nv_bfloat16*)qkv,
+        e = launch(fixed_decay_output_kernel, dim3((unsigned)bx, nh, num_seqs), FD_CT, smem, stream, (const __nv_bfloat16*)qkv,
                    qkv_stride, q_off, k_off, v_off, powers, q_scale, act, state_slots, cu_q, positions, (const uint4*)scratch,
                    scratch_chunks, out, nh, rows, cols, num_slots, min_q);
         rc = check_launch("fixed_decay (output)", e);

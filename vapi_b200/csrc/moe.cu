@@ -50,60 +50,79 @@ template <> struct RtLd4<__nv_bfloat16> {
     }
 };
 
-// One block of four warps per token: the warps share the router's outputs among them (four outputs at a time
-// a warp, so that a lane has their loads in flight together), then the first warp chooses.  The order of a
-// lane's additions and of a warp's reduction depends on nothing but the width.  shared memory: 2 * outputs
-// floats (the scores and the choice scores) + groups floats + one (the shared expert's gate).
-template <typename T>
-__global__ void __launch_bounds__(128)
+// A block takes TPB tokens (one in small steps; four in prompts, so that a row of the router is read once for four
+// tokens).  The warps share the router's outputs among them (four outputs at a time a warp, so that a lane has their
+// loads in flight together), then a warp per token chooses.  The order of a lane's additions and of a warp's reduction
+// depends on nothing but the width.  shared memory per token: 2 * outputs floats (the scores and the choice scores) +
+// groups floats + one (the shared expert's gate).
+constexpr int RT_MAX_WARPS = 16;
+template <typename T, int TPB>
+__global__ void __launch_bounds__(RT_MAX_WARPS * 32)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ corr,
                  const float* __restrict__ bias, int score_mode,
                  int* __restrict__ ids, float* __restrict__ wts, int n, int width, int outputs, int experts, int top,
                  int groups, int keep, int vec4, int group_top, float* __restrict__ shared_gate) {
     extern __shared__ float rt_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-    const int t = blockIdx.x;
-    float* s = rt_smem;
+    const int t_first = blockIdx.x * TPB;
     const int nrows = outputs + (shared_gate ? 1 : 0);         // the router's rows, and the shared expert's gate
-    float* choice = s + outputs + 1;
-    float* gscore = choice + outputs;
+    const int per_token = 2 * outputs + groups + 1;            // floats of shared memory
     pdl_trigger();
     pdl_wait();
-    if (t >= n) return;
-    const T* hr = h + (size_t)t * width;
     for (int e0 = warp * 4; e0 < nrows; e0 += warps * 4) {
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
-        const float* w0 = wr + (size_t)e0 * width;
+        float acc[4][TPB];
+        const float* w0[4];
+        const T* hr[TPB];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            w0[j] = wr + (size_t)min(e0 + j, nrows - 1) * width;                   // (a row that does not exist is not stored)
+#pragma unroll
+            for (int u = 0; u < TPB; ++u) acc[j][u] = 0.f;
+        }
+#pragma unroll
+        for (int u = 0; u < TPB; ++u) hr[u] = h + (size_t)min(t_first + u, n - 1) * width;
         if (vec4) {
+#pragma unroll (TPB == 1 ? 4 : 2)
             for (int k = lane * 4; k < width; k += 128) {
-                const float4 hv = RtLd4<T>::load(hr + k);
+                float4 hv[TPB];
+#pragma unroll
+                for (int u = 0; u < TPB; ++u) hv[u] = RtLd4<T>::load(hr[u] + k);
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
-                    if (e0 + j < nrows) {
-                        const float4 wv = *reinterpret_cast<const float4*>(w0 + (size_t)j * width + k);
-                        acc[j] = fmaf(hv.x, wv.x, acc[j]);
-                        acc[j] = fmaf(hv.y, wv.y, acc[j]);
-                        acc[j] = fmaf(hv.z, wv.z, acc[j]);
-                        acc[j] = fmaf(hv.w, wv.w, acc[j]);
+                    const float4 wv = *reinterpret_cast<const float4*>(w0[j] + k);
+#pragma unroll
+                    for (int u = 0; u < TPB; ++u) {
+                        acc[j][u] = fmaf(hv[u].x, wv.x, acc[j][u]);
+                        acc[j][u] = fmaf(hv[u].y, wv.y, acc[j][u]);
+                        acc[j][u] = fmaf(hv[u].z, wv.z, acc[j][u]);
+                        acc[j][u] = fmaf(hv[u].w, wv.w, acc[j][u]);
                     }
                 }
             }
         } else {
             for (int k = lane; k < width; k += 32) {
-                const float hv = to_f32(hr[k]);
 #pragma unroll
-                for (int j = 0; j < 4; ++j)
-                    if (e0 + j < nrows) acc[j] = fmaf(hv, w0[(size_t)j * width + k], acc[j]);
+                for (int u = 0; u < TPB; ++u) {
+                    const float hv = to_f32(hr[u][k]);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) acc[j][u] = fmaf(hv, w0[j][k], acc[j][u]);
+                }
             }
         }
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const float v = warp_sum(acc[j]);
-            if (lane == 0 && e0 + j < nrows) s[e0 + j] = bias && e0 + j < outputs ? v + bias[e0 + j] : v;
-        }
+        for (int u = 0; u < TPB; ++u)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float v = warp_sum(acc[j][u]);
+                if (lane == 0 && e0 + j < nrows) rt_smem[u * per_token + e0 + j] = bias && e0 + j < outputs ? v + bias[e0 + j] : v;
+            }
     }
     __syncthreads();
-    if (warp != 0) return;
+    if (warp >= TPB || t_first + warp >= n) return;
+    const int t = t_first + warp;
+    float* s = rt_smem + warp * per_token;
+    float* choice = s + outputs + 1;
+    float* gscore = choice + outputs;
     {
 
     __syncwarp();
@@ -468,6 +487,40 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
     }
 }
 
+// The same with four columns a thread (width a multiple of 4, 16-byte / 8-byte aligned rows).
+template <typename T> struct RtSt4;
+template <> struct RtSt4<float> {
+    static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+};
+template <> struct RtSt4<__nv_bfloat16> {
+    static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
+};
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(const float* __restrict__ y, const int* __restrict__ ids, const float* __restrict__ wts,
+                       const T* __restrict__ h, const T* __restrict__ shared, T* __restrict__ out, int n, int width, int top,
+                       int experts, const float* __restrict__ shared_gate) {
+    const int t = blockIdx.x, c = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+    pdl_trigger();
+    pdl_wait();
+    if (t >= n || c >= width) return;
+    const size_t at = (size_t)t * width + c;
+    const float4 sh = shared ? RtLd4<T>::load(shared + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float gate = shared_gate ? shared_gate[t] : 1.f;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int r = 0; r < top; ++r) {
+        const size_t p = (size_t)t * top + r;
+        float4 v;
+        float g = 1.f;
+        if (ids[p] < experts) v = *reinterpret_cast<const float4*>(y + p * width + c);
+        else { v = RtLd4<T>::load(h + at); g = wts[p]; }
+        acc.x += g * v.x; acc.y += g * v.y; acc.z += g * v.z; acc.w += g * v.w;
+    }
+    if (shared) { acc.x = fmaf(gate, sh.x, acc.x); acc.y = fmaf(gate, sh.y, acc.y); acc.z = fmaf(gate, sh.z, acc.z); acc.w = fmaf(gate, sh.w, acc.w); }
+    RtSt4<T>::store(out + at, acc);
+}
+
 template <typename T>
 __global__ void relu_squared_kernel(const T* __restrict__ x, T* __restrict__ out, long long total) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -526,15 +579,19 @@ VAPI_EXPORT int vapi_moe_route(const void* h, int dtype, const float* wr, const 
         return fail(-1, "moe_route: %d outputs in %d groups, %d kept", outputs, groups, keep);
     if ((long long)(outputs / groups) * keep < top) return fail(-1, "moe_route: %d kept groups cannot give %d choices", keep, top);
     cudaError_t e;
-    const size_t smem = (size_t)(2 * outputs + groups + 1) * sizeof(float);
+    const int rows = outputs + (shared_gate ? 1 : 0);
+    const int tpb = n >= 1024 && 2 * outputs + groups + 1 <= 3000 ? 4 : 1;
+    const int warps = max(tpb, min(RT_MAX_WARPS, (rows + 3) / 4));
+    const int blocks = (n + tpb - 1) / tpb;
+    const size_t smem = (size_t)tpb * (2 * outputs + groups + 1) * sizeof(float);
     if (smem > 48 * 1024) return fail(-1, "moe_route: %d router outputs are too many", outputs);
     const int vec4 = (width % 4 == 0 && ((uintptr_t)h & 15) == 0 && ((uintptr_t)wr & 15) == 0) ? 1 : 0;
-    if (dtype == VAPI_F32)
-        e = launch(moe_route_kernel<float>, n, 128, smem, stream, (const float*)h, wr, corr, bias, score_mode, ids, wts, n,
-                   width, outputs, experts, top, groups, keep, vec4, group_top, shared_gate);
-    else if (dtype == VAPI_BF16)
-        e = launch(moe_route_kernel<__nv_bfloat16>, n, 128, smem, stream, (const __nv_bfloat16*)h, wr, corr, bias, score_mode, ids,
-                   wts, n, width, outputs, experts, top, groups, keep, vec4, group_top, shared_gate);
+#define RT_GO(T, B)                                                                                                           \
+    e = launch(moe_route_kernel<T, B>, blocks, warps * 32, smem, stream, (const T*)h, wr, corr, bias, score_mode, ids, wts, n,  \
+               width, outputs, experts, top, groups, keep, vec4, group_top, shared_gate)
+    if (dtype == VAPI_F32) { if (tpb == 4) RT_GO(float, 4); else RT_GO(float, 1); }
+    else if (dtype == VAPI_BF16) { if (tpb == 4) RT_GO(__nv_bfloat16, 4); else RT_GO(__nv_bfloat16, 1); }
+#undef RT_GO
     else
         return fail(-2, "moe_route: unsupported dtype %d", dtype);
     int rc = check_launch("moe_route", e);
@@ -616,6 +673,18 @@ VAPI_EXPORT int vapi_moe_combine(const float* y, const int* ids, const float* wt
     if (n <= 0) return 0;
     const int threads = width >= 1024 ? 256 : 128;
     cudaError_t e;
+    const size_t ends = (size_t)(((uintptr_t)y) & 15) | (((uintptr_t)h | (uintptr_t)shared | (uintptr_t)out) & (dtype == VAPI_F32 ? 15 : 7));
+    if (width % 4 == 0 && ends == 0 && (dtype == VAPI_F32 || dtype == VAPI_BF16)) {
+        const int th = width >= 1024 ? 256 : ((width / 4 + 31) / 32) * 32;
+        dim3 grid(n, (width / 4 + th - 1) / th);
+        if (dtype == VAPI_F32)
+            e = launch(moe_combine_vec_kernel<float>, grid, th, 0, stream, y, ids, wts, (const float*)h, (const float*)shared,
+                       (float*)out, n, width, top, experts, shared_gate);
+        else
+            e = launch(moe_combine_vec_kernel<__nv_bfloat16>, grid, th, 0, stream, y, ids, wts, (const __nv_bfloat16*)h,
+                       (const __nv_bfloat16*)shared, (__nv_bfloat16*)out, n, width, top, experts, shared_gate);
+        return check_launch("moe_combine", e);
+    }
     if (dtype == VAPI_F32)
         e = launch(moe_combine_kernel<float>, n, threads, 0, stream, y, ids, wts, (const float*)h, (const float*)shared,
                    (float*)out, n, width, top, experts, shared_gate);
