@@ -32,7 +32,8 @@ def folders(tmp_path_factory):
     for name, cfg, seed in [("mixed", zu.MIXED, 1), ("tiny", zu.TINY, 2), ("plain", zu.PLAIN, 3), ("serving_heads", zu.SERVING_HEADS, 4)] + \
             [(k, v, 10 + i) for i, (k, v) in enumerate(zu.ONE.items())]:
         out[name] = zu.write_model(str(tmp_path_factory.mktemp(name)), cfg, seed)
-        out[name + "/bf16"] = zu.write_model(str(tmp_path_factory.mktemp(name + "bf16")), cfg, seed, torch.bfloat16, planted_routes=True)
+        out[name + "/bf16"] = zu.write_model(str(tmp_path_factory.mktemp(name + "bf16")), zu.PLAIN_16 if name == "plain" else cfg, seed, torch.bfloat16,
+                                             planted_routes=True)
     return out
 
 
@@ -216,7 +217,8 @@ BATCH = [pytest.param("cpu", "tiny", "float32", [7, 1, 12, 3, 9], 16, id="host")
          pytest.param("cuda", "mixed", "float32", [70, 1, 33, 150, 2, 64, 17], 16, marks=pytest.mark.gpu, id="gpu-f32"),
          pytest.param("cuda", "mixed/bf16", "bfloat16", [70, 1, 33, 150, 2, 64, 17], 16, marks=pytest.mark.gpu, id="gpu-bf16"),
          pytest.param("cuda", "serving_heads/bf16", "bfloat16", [150, 40, 3, 86, 170], 64, marks=pytest.mark.gpu, id="gpu-bf16-tensor-cores"),
-         pytest.param("cuda", "retention/bf16", "bfloat16", [60, 5, 31], 16, marks=pytest.mark.gpu, id="gpu-bf16-retention")]
+         pytest.param("cuda", "retention/bf16", "bfloat16", [60, 5, 31], 16, marks=pytest.mark.gpu, id="gpu-bf16-retention"),
+         pytest.param("cuda", "plain/bf16", "bfloat16", [60, 5, 31], 16, marks=pytest.mark.gpu, id="gpu-bf16-plain")]
 
 
 @pytest.mark.parametrize("device,name,dtype,lens,page", BATCH)

@@ -69,6 +69,10 @@ PLAIN = config([layer(memory("lightning", heads=1, dim=16, vdim=16, decay=[1.0])
                 layer(memory("retention", heads=1, dim=1, vdim=3, decay=[1e-3]), moe(ff=10, experts=4, top=4, groups=(4, 4), shared=6)),
                 layer(attention(heads=2, kv_heads=2, dim=8, vdim=8, size=None, dims=2, base=1.5, scaling=(2.0, 0.5, 0.5, 9.0)), None),
                 layer(memory("retention", heads=3, dim=7, vdim=5, decay=[1.0, 0.0, 0.9]), dense(33))], width=66, vocab=91)
+#: the same for bfloat16: a head of one key element that forgets at once reads nothing but the sign of q times k, which is no
+#: matter of rounding
+PLAIN_16 = config(PLAIN["layers"][:2] + [layer(memory("retention", heads=1, dim=9, vdim=3, decay=[0.95]), PLAIN["layers"][2]["mlp"])] + PLAIN["layers"][3:4],
+                  width=66, vocab=91)
 #: sizes of the serving kernels (the tensor cores for bfloat16: head sizes of 64 and 128 in the attention, states that the
 #: chunked form takes, also with padding on both sides)
 SERVING_HEADS = config([layer(attention(heads=6, kv_heads=2, dim=64, vdim=64, scale=0.12, size=90, dims=48, base=1e4, scaling=(4.0, 1.0, 4.0, 64.0)), dense(160)),

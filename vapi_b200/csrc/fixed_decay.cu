@@ -77,7 +77,8 @@ __device__ __forceinline__ float4 fd_act4(float4 v, int act) {
     return v;
 }
 
-template <typename T, int RPL, int LPC, int NC>
+// TG: tokens in flight (one in decode steps: fewer registers, more warps with their part of a state under way)
+template <typename T, int RPL, int LPC, int NC, int TG>
 __global__ void __launch_bounds__(FD_THREADS)
 fixed_decay_walk_kernel(const T* __restrict__ qkv, long long qkv_stride, int q_off, int k_off, int v_off,
                         const float* __restrict__ powers, float q_scale, int act, float* __restrict__ state, long long slot_stride,
@@ -85,7 +86,6 @@ fixed_decay_walk_kernel(const T* __restrict__ qkv, long long qkv_stride, int q_o
                         float* __restrict__ out, int nh, int rows, int cols, int num_slots, int q_below, int wide,
                         int* __restrict__ status) {
     static_assert(RPL % 4 == 0 && NC % 4 == 0 && NC <= LPC, "rows and columns of a lane come in fours");
-    constexpr int TG = sizeof(T) == 4 ? 2 : 4;                          // tokens in flight
     constexpr int GROUPS = 32 / LPC;
     const int s = blockIdx.z, h = blockIdx.y;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -594,10 +594,11 @@ VAPI_EXPORT int vapi_fixed_decay(const void* qkv, long long qkv_stride, int q_of
     const int q_below = chunked ? min_q : 0;
     cudaError_t e = cudaSuccess;
     const bool early = max_q < 16;
-#define FD_WALK(T, RPL, LPC, NC)                                                                                              \
-    e = launch_if(early, fixed_decay_walk_kernel<T, RPL, LPC, NC>, dim3((cols + (32 / LPC) * NC * 4 - 1) / ((32 / LPC) * NC * 4), nh, num_seqs), \
+#define FD_WALK_(T, RPL, LPC, NC, TG)                                                                                         \
+    e = launch_if(early, fixed_decay_walk_kernel<T, RPL, LPC, NC, TG>, dim3((cols + (32 / LPC) * NC * 4 - 1) / ((32 / LPC) * NC * 4), nh, num_seqs), \
                   FD_THREADS, 0, stream, (const T*)qkv, qkv_stride, q_off, k_off, v_off, powers, q_scale, act, state,         \
                   slot_stride, state_slots, cu_q, positions, out, nh, rows, cols, num_slots, q_below, wide, status)
+#define FD_WALK(T, RPL, LPC, NC) do { if (max_q == 1) FD_WALK_(T, RPL, LPC, NC, 1); else FD_WALK_(T, RPL, LPC, NC, sizeof(T) == 4 ? 2 : 4); } while (0)
 #define FD_SIZES(T)                                                                                                           \
     do {                                                                                                                      \
         if (rows <= 32) FD_WALK(T, 4, 8, 4);                                                                                  \
@@ -610,6 +611,7 @@ VAPI_EXPORT int vapi_fixed_decay(const void* qkv, long long qkv_stride, int q_of
     else FD_SIZES(__nv_bfloat16);
 #undef FD_SIZES
 #undef FD_WALK
+#undef FD_WALK_
     return check_launch("fixed_decay (walk)", e);
 }
 

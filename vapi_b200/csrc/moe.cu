@@ -82,7 +82,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const fl
 #pragma unroll
         for (int u = 0; u < TPB; ++u) hr[u] = h + (size_t)min(t_first + u, n - 1) * width;
         if (vec4) {
-#pragma unroll (TPB == 1 ? 4 : 2)
+#pragma unroll (TPB == 1 ? 4 : 1)
             for (int k = lane * 4; k < width; k += 128) {
                 float4 hv[TPB];
 #pragma unroll
